@@ -4,6 +4,7 @@ from .falalix import FalalixConfig
 from .govopel import GovopelConfig
 from .navulorn import NavulornConfig
 from .qwen3 import Qwen3Config
+from .rusolorn import RusolornConfig
 from .registry import (config_class, config_from_dict, load_config, register_architecture,
                        supported_architectures)
 
@@ -12,7 +13,8 @@ register_architecture("Falalix", FalalixConfig)
 register_architecture("Govopel", GovopelConfig)
 register_architecture("Divuzen", DivuzenConfig)
 register_architecture("Navulorn", NavulornConfig)
+register_architecture("Rusolorn", RusolornConfig)
 
-__all__ = ["ConfigError", "LayerSpec", "ModelConfig", "ModelSpec", "PartSpec", "RunEntry", "Qwen3Config", "FalalixConfig", "GovopelConfig", "DivuzenConfig", "NavulornConfig",
+__all__ = ["ConfigError", "LayerSpec", "ModelConfig", "ModelSpec", "PartSpec", "RunEntry", "Qwen3Config", "FalalixConfig", "GovopelConfig", "DivuzenConfig", "NavulornConfig", "RusolornConfig",
            "config_class", "config_from_dict", "load_config", "register_architecture",
            "supported_architectures"]

@@ -39,6 +39,7 @@ class LayerSpec:
     norms: Mapping[str, PartSpec]
     position: Optional[PartSpec] = None
     block_params: Mapping[str, Any] = field(default_factory=dict)    # constants of the arrangement itself
+    side: Optional[PartSpec] = None  # something more that joins the stream behind the sublayers (category 'side')
 
 
 @dataclass(frozen=True)

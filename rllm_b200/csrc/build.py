@@ -31,8 +31,9 @@ NVCC_FLAGS = [
 
 # library name -> (sources, extra link flags)
 LIBRARIES = {
-    "core": (["elementwise.cu", "rowwise.cu", "headwise.cu", "attention_generic.cu", "gemm_plain.cu", "sampling.cu"], []),
+    "core": (["elementwise.cu", "rowwise.cu", "headwise.cu", "joins.cu", "attention_generic.cu", "gemm_plain.cu", "sampling.cu"], []),
     "recur": (["recurrent.cu"], []),
+    "delta": (["delta.cu"], []),
     "moe": (["moe.cu"], []),
     "blas": (["gemm_lib.cu"], ["-lcublas"]),
     "fast": (["skinny_gemm.cu"], []),

@@ -437,6 +437,76 @@ def sum_norm_rows(x, y, alpha, weight, eps, low=None):
     return x
 
 
+# ------------------------------------------------------------------ side-by-side sublayers, Dynamic Tanh, token table (joins.cu)
+
+def dyt_rows(x, alpha, weight, bias, out, delta=None, delta_scale=1.0, rows=None, write_x=True):
+    """out[r] = tanh(alpha * v) * weight + bias, v = x[src] (+ delta_scale * delta[src]), src = rows[r] if rows
+    is given else r; x (the float32 stream) receives the sum when write_x and delta is given."""
+    _need_cuda(x, delta, weight, bias, out, rows)
+    _need_contig(x=x, delta=delta, weight=weight, bias=bias, out=out, rows=rows)
+    n, d = out.shape
+    assert x.dtype == torch.float32 and x.shape[1] == d and (rows is not None or x.shape[0] == n)
+    assert weight.dtype == bias.dtype == torch.float32 and weight.numel() == bias.numel() == d
+    assert rows is None or (rows.dtype == torch.int32 and rows.numel() == n)
+    assert delta is None or (delta.dtype == torch.float32 and delta.shape == x.shape)
+    _check(core().rllm_dyt_rows(_ptr(x), _ptr(delta), c_float(delta_scale), _ptr(rows), c_float(alpha), _ptr(weight),
+                                _ptr(bias), _ptr(out), c_int(_code(out)), c_int(n), c_int(d), c_int(1 if write_x else 0),
+                                _stream()), "dyt_rows")
+    return out
+
+
+def join_sum_rows(a, x, mult=1.0, add=True, norm_a=None, scale_a=1.0, b=None, norm_b=None, scale_b=1.0, c=None, low=None):
+    """x (+)= mult * (scale_a * N_a(a) + scale_b * N_b(b) + c) over float32 rows; norm_a, norm_b: (weight, eps) of
+    an RMS norm or None for the rows themselves; b, c optional; `low` (optional) takes x in its own type.  add
+    False: x is written, its old rows are not read."""
+    _need_cuda(a, x, b, c, low)
+    _need_contig(x=x, low=low)
+    n, d = x.shape
+    for name, t in (("a", a), ("b", b), ("c", c)):
+        assert t is None or (_rows2d(t, name).shape == (n, d) and t.dtype == torch.float32)
+    assert x.dtype == torch.float32 and (low is None or low.shape == (n, d)) and (b is not None or norm_b is None)
+    for nm in (norm_a, norm_b):
+        assert nm is None or (nm[0].dtype == torch.float32 and nm[0].numel() == d and nm[0].is_contiguous())
+    wa, ea = norm_a or (None, 0.0)
+    wb, eb = norm_b or (None, 0.0)
+    st = lambda t: c_longlong(t.stride(0) if t is not None else 0)
+    _check(core().rllm_join_sum_rows(_ptr(a), st(a), _ptr(wa), c_float(ea), c_float(scale_a), _ptr(b), st(b), _ptr(wb),
+                                     c_float(eb), c_float(scale_b), _ptr(c), st(c), c_float(mult), _ptr(x),
+                                     c_int(1 if add else 0), _ptr(low), c_int(_code(low) if low is not None else F32),
+                                     c_int(n), c_int(d), _stream()), "join_sum_rows")
+    return x
+
+
+def join_dyt_rows(y, norm_y, mult, x, alpha, weight, bias, out):
+    """x += mult * y / rms(y) * w with norm_y = (w, eps), and in the same kernel out = tanh(alpha * x) * weight + bias
+    of the new x."""
+    _need_cuda(y, x, weight, bias, out, norm_y[0])
+    _need_contig(x=x, weight=weight, bias=bias, out=out)
+    n, d = x.shape
+    wy, eps = norm_y
+    assert x.dtype == y.dtype == torch.float32 and _rows2d(y, "y").shape == (n, d) and out.shape == (n, d)
+    for w in (wy, weight, bias):
+        assert w.dtype == torch.float32 and w.numel() == d and w.is_contiguous()
+    _check(core().rllm_join_dyt_rows(_ptr(y), c_longlong(y.stride(0)), _ptr(wy), c_float(eps), c_float(mult), _ptr(x),
+                                     c_float(alpha), _ptr(weight), _ptr(bias), _ptr(out), c_int(_code(out)), c_int(n),
+                                     c_int(d), _stream()), "join_dyt_rows")
+    return out
+
+
+def token_gate(z, table, tokens, out, dim):
+    """out[t, c] = gelu_tanh(z[t, c]) * table[tokens[t], c] for c < dim, 0 in the columns behind (padding);
+    z float32 (any row stride), table [vocab, dim] and out of one type."""
+    _need_cuda(z, table, tokens, out)
+    _need_contig(table=table, tokens=tokens, out=out)
+    n, padded = out.shape
+    assert z.dtype == torch.float32 and _rows2d(z, "z").shape[0] == n and z.shape[1] >= dim and padded >= dim
+    assert table.shape[1] == dim and table.dtype == out.dtype and tokens.dtype == torch.int32 and tokens.numel() == n
+    _check(core().rllm_token_gate(_ptr(z), c_longlong(z.stride(0)), _ptr(table), _ptr(tokens), _ptr(out), c_int(_code(out)),
+                                  c_int(n), c_int(dim), c_int(padded), c_int(table.shape[0]), _ptr(error_word(z.device)),
+                                  _stream()), "token_gate")
+    return out
+
+
 def rope_unitnorm_store(rows, cs_table, rot, cs_mult, slots, q_out, k_cache, v_cache, H, G, hd, block_size, eps,
                         unit_norm=True, v_tied=True, write_kv=True):
     """rows [n, (H + G) * hd (+ G * hd values)] -> per head: the first `rot` entries rotated by the
@@ -610,18 +680,20 @@ def cat2_cast(x, y, out, delta=None, delta_scale=1.0):
 
 
 def qkv_rownorm_store(qkv, bias, q_norm_w, k_norm_w, slots, q_out, k_cache, v_cache, H, G, dk, dv, block_size, eps,
-                      write_kv=True, cs_table=None, rot=0, pairs=False):
+                      write_kv=True, cs_table=None, rot=0, pairs=False, v_tied=False):
     """Biased q/k/v row -> RMSNorm over the whole q row and the whole k row (weights per column, None:
     no norm) -> with `rot` > 0 the first rot entries of every query and key head rotated by the angles of
     cs_table [n, rot/2, 2] (entry i with i + rot/2, or 2i with 2i + 1 when `pairs`) -> queries out, keys and
-    values into the paged cache; see rowwise.cu."""
+    values into the paged cache; see rowwise.cu.  v_tied: the rows are [q | k] and the values are the key
+    columns as projected (before the norm)."""
     _need_cuda(qkv, bias, q_norm_w, k_norm_w, slots, q_out, k_cache, v_cache, cs_table)
     assert rot == 0 or (cs_table.dtype == torch.float32 and cs_table.shape == (qkv.shape[0], rot // 2, 2)
                         and cs_table.is_contiguous() and rot % 2 == 0 and rot <= dk)
     _need_contig(q_out=q_out, k_cache=k_cache, v_cache=v_cache, slots=slots)
     _rows2d(qkv, "qkv")                       # may be the leading columns of a wider projection
     n = qkv.shape[0]
-    assert qkv.shape[1] == H * dk + G * dk + G * dv and q_out.shape == (n, H * dk)
+    assert qkv.shape[1] == H * dk + G * dk + (0 if v_tied else G * dv) and q_out.shape == (n, H * dk)
+    assert not v_tied or dv == dk
     assert slots.dtype == torch.int32 and slots.numel() == n
     assert k_cache.shape[1:] == (G, block_size, dk) and v_cache.shape[1:] == (G, block_size, dv)
     assert k_cache.dtype == v_cache.dtype == q_out.dtype
@@ -632,7 +704,8 @@ def qkv_rownorm_store(qkv, bias, q_norm_w, k_norm_w, slots, q_out, k_cache, v_ca
         _ptr(slots), _ptr(q_out),
         _ptr(k_cache), _ptr(v_cache), c_int(_code(q_out)), c_int(n), c_int(H), c_int(G), c_int(dk), c_int(dv),
         c_int(block_size), c_float(eps), c_int(1 if write_kv else 0), c_longlong(k_cache.shape[0] * block_size),
-        _ptr(error_word(qkv.device)), _ptr(cs_table if rot else None), c_int(rot), c_int(1 if pairs else 0), _stream()),
+        _ptr(error_word(qkv.device)), _ptr(cs_table if rot else None), c_int(rot), c_int(1 if pairs else 0),
+        c_int(H * dk if v_tied else (H + G) * dk), _stream()),
         "qkv_rownorm_store")
     return q_out
 
@@ -900,6 +973,53 @@ def mlstm(rows, q_off, k_off, v_off, g_off, i_off, f_off, i_bias, f_bias, cap, q
     if sg is not None:
         global _launches
         _launches += 2                         # the local pass and the combine kernel
+    return out
+
+
+DELTA_STEP_TOKENS = 8         # steps in which no request brings more tokens than this take the token-by-token kernel
+
+
+def delta_state_floats(H: int, dk: int, dv: int, taps: int) -> int:
+    """Floats of a request's gated-delta state: per head the dk x dv memory padded to the kernels' tile and in
+    their threads' order, then per head the kept inputs of its convolutions (delta.cu).  No device needed."""
+    DK = next(s for s in (32, 64, 128, 256, 512) if dk <= s)
+    return H * DK * (-(-dv // 8) * 8) + H * (2 * dk + dv) * (taps - 1)
+
+
+def gated_delta(rows, offs, conv, A, dt_bias, norm_w, q_scale, unit_eps, eps, state, cu_q, slots, out, n_requests, max_q_len,
+                H, G, dk, dv, gate="silu"):
+    """The gated delta rule with its convolutions, unit vectors, gates and output norm over each request's
+    tokens, its state in state[slot]; see delta.cu.  rows: float32 [n, ...] with q, k ([G*dk] each), v, gate
+    ([H*dv] each), b and a ([H] each) at the column offsets `offs` in this order; conv float32 [2 G dk + H dv, taps]; A,
+    dt_bias float32 [H]; norm_w float32 [dv]; out activation type [n, H*dv].  max_q_len: the most tokens a
+    request brings in this step (it decides between the token-by-token kernel and the chunked ones)."""
+    _need_cuda(rows, conv, A, dt_bias, norm_w, state, cu_q, slots, out)
+    _rows2d(rows, "rows")
+    _need_contig(out=out, conv=conv, A=A, dt_bias=dt_bias, norm_w=norm_w)
+    n, taps = out.shape[0], conv.shape[1]
+    assert rows.dtype == torch.float32 and rows.shape[0] == n and out.shape == (n, H * dv) and H % G == 0
+    for off, size in zip(offs, (G * dk, G * dk, H * dv, H * dv, H, H)):
+        assert off + size <= rows.shape[1]
+    assert conv.shape[0] == 2 * G * dk + H * dv and A.numel() == dt_bias.numel() == H and norm_w.numel() == dv
+    assert conv.dtype == A.dtype == dt_bias.dtype == norm_w.dtype == torch.float32
+    if dk > 512 or taps > 64:
+        raise KernelError(f"gated_delta: key heads up to 512 entries and up to 64 taps, got {dk} and {taps}")
+    st = _state2d(state)
+    assert delta_state_floats(H, dk, dv, taps) <= st.shape[1]
+    portion = max_q_len > DELTA_STEP_TOKENS
+    new = lambda *s: torch.empty(s, dtype=torch.float32, device=out.device)
+    qn = kn = prods = bg = o = None
+    if portion:
+        qn, kn, prods, bg, o = new(n, G * dk), new(n, G * dk), new(n, G, 16), new(n, H, 2), new(n, H * dv)
+    _check(_lib("delta").rllm_gated_delta(
+        _ptr(rows), c_longlong(rows.stride(0)), *(c_int(x) for x in offs), _ptr(conv), _ptr(A), _ptr(dt_bias), _ptr(norm_w),
+        c_float(q_scale), c_float(unit_eps), c_float(eps), _ptr(st), c_longlong(st.stride(0)), _ptr(cu_q), _ptr(slots),
+        _ptr(out), c_int(_code(out)), c_int(n), c_int(n_requests), c_int(H), c_int(G), c_int(dk), c_int(dv), c_int(taps),
+        c_int(GATES[gate]), c_int(1 if portion else 0), _ptr(qn), _ptr(kn), _ptr(prods), _ptr(bg), _ptr(o), _stream()),
+        "gated_delta")
+    if portion:
+        global _launches
+        _launches += 2                         # prep, chunk and out
     return out
 
 

@@ -20,10 +20,7 @@
 //           four floats of which the first is the running maximum m.  Heads beyond the kernel's sizes: S
 //           [dk][dv + 1] row-major and the four floats.
 #include "common.cuh"
-#include <math.h>
-
-__device__ __forceinline__ float silu_f(float z) { return z / (1.0f + expf(-z)); }
-__device__ __forceinline__ float softplus_f(float z) { return z > 20.f ? z : log1pf(expf(z)); }
+#include "recurrent.cuh"
 
 // ------------------------------------------------------------------ causal convolution + silu
 // xz [n, ld] float32 holds the convolution's input in columns [0, inner).  Token t (index i in

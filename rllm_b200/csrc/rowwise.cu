@@ -8,7 +8,8 @@
 //   qkv_rownorm_store  biased q/k/v projection row -> RMSNorm over the WHOLE q row and the whole k
 //                   row (one weight per column), then optionally the rotation of the first `rot` entries
 //                   of every query and key head by the step's angles; queries out, keys and values into
-//                   the paged cache; the value heads may have another size than the key heads
+//                   the paged cache; the value heads may have another size than the key heads, or the
+//                   values are the key columns as projected (v_off = the keys' first column)
 //
 // f1, f2: 0 identity, 1 silu z / (1 + e^-z), 2 relu(z)^2, 3 sigmoid, 4 tanh, 5 softplus.
 #include "common.cuh"
@@ -137,7 +138,7 @@ __global__ void __launch_bounds__(1024)
 qkv_rownorm_store_kernel(const TI* qkv, const float* __restrict__ bias, const float* __restrict__ q_norm_w,
                          const float* __restrict__ k_norm_w, const int* __restrict__ slots, TO* q_out, TO* k_cache,
                          TO* v_cache, long long ld, int wq, int wk, int wv, int G, int dk, int dv, int bs, float eps,
-                         int write_kv, int n_slots, int* err, const float2* cs_table, int rot, int pairs) {
+                         int write_kv, int n_slots, int* err, const float2* cs_table, int rot, int pairs, int v_off) {
     __shared__ float red[33];
     extern __shared__ float staged_row[];
     pdl_launch_dependents();
@@ -192,7 +193,7 @@ qkv_rownorm_store_kernel(const TI* qkv, const float* __restrict__ bias, const fl
     for (int c = tid; c < wk; c += blockDim.x)
         k_cache[((page * G + c / dk) * bs + off) * dk + c % dk] = from_f<TO>(turned(wq, c, k_norm_w, rk));
     for (int c = tid; c < wv; c += blockDim.x) {
-        const float v = to_f<TI>(row[wq + wk + c]) + (bias ? bias[wq + wk + c] : 0.f);
+        const float v = to_f<TI>(row[v_off + c]) + (bias ? bias[v_off + c] : 0.f);
         v_cache[((page * G + c / dv) * bs + off) * dv + c % dv] = from_f<TO>(v);
     }
 }
@@ -201,9 +202,10 @@ RLLM_API int rllm_qkv_rownorm_store(const void* qkv, int in_dt, long long ld, co
                                     const float* k_norm_w, const int* slots, void* q_out, void* k_cache,
                                     void* v_cache, int out_dt, int n, int H, int G, int dk, int dv, int bs,
                                     float eps, int write_kv, long long n_slots, int* err, const void* cs_table,
-                                    int rot, int pairs, cudaStream_t stream) {
+                                    int rot, int pairs, int v_off, cudaStream_t stream) {
     if (n <= 0) return 0;
-    if (H <= 0 || G <= 0 || dk <= 0 || dv <= 0 || bs <= 0 || ld < (long long)H * dk + (long long)G * (dk + dv) ||
+    if (H <= 0 || G <= 0 || dk <= 0 || dv <= 0 || bs <= 0 || v_off < 0 || ld < (long long)v_off + (long long)G * dv ||
+        ld < (long long)(H + G) * dk ||
         rot < 0 || rot > dk || (rot & 1) || (rot && !cs_table))
         return (int)cudaErrorInvalidValue;
     const int ns = (int)(n_slots > 0x7fffffffLL ? 0x7fffffffLL : n_slots);
@@ -214,10 +216,10 @@ RLLM_API int rllm_qkv_rownorm_store(const void* qkv, int in_dt, long long ld, co
     if (smem <= 40 * 1024)                                                                                     \
         return rllm_launch(qkv_rownorm_store_kernel<TI, TO, true>, dim3(n), dim3(threads), smem, stream, (const TI*)qkv, \
                            bias, q_norm_w, k_norm_w, slots, (TO*)q_out, (TO*)k_cache, (TO*)v_cache, ld, H * dk, G * dk, \
-                           G * dv, G, dk, dv, bs, eps, write_kv, ns, err, (const float2*)cs_table, rot, pairs);    \
+                           G * dv, G, dk, dv, bs, eps, write_kv, ns, err, (const float2*)cs_table, rot, pairs, v_off);    \
     return rllm_launch(qkv_rownorm_store_kernel<TI, TO, false>, dim3(n), dim3(threads), 0, stream, (const TI*)qkv, bias, \
                        q_norm_w, k_norm_w, slots, (TO*)q_out, (TO*)k_cache, (TO*)v_cache, ld, H * dk, G * dk, G * dv, \
-                       G, dk, dv, bs, eps, write_kv, ns, err, (const float2*)cs_table, rot, pairs)
+                       G, dk, dv, bs, eps, write_kv, ns, err, (const float2*)cs_table, rot, pairs, v_off)
     if (in_dt == RLLM_F32 && out_dt == RLLM_F32) { LAUNCH(float, float); }
     if (in_dt == RLLM_F32 && out_dt == RLLM_BF16) { LAUNCH(float, bf16); }
     if (in_dt == RLLM_BF16 && out_dt == RLLM_BF16) { LAUNCH(bf16, bf16); }

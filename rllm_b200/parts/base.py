@@ -14,7 +14,7 @@ from typing import Any, Callable, Mapping, Optional
 
 import torch
 
-CATEGORIES = ("embedding", "norm", "position", "mixer", "ffn", "block", "lm_head", "junction")
+CATEGORIES = ("embedding", "norm", "position", "mixer", "ffn", "block", "lm_head", "junction", "side")
 _REGISTRY: dict[str, dict[str, Callable]] = {c: {} for c in CATEGORIES}
 
 
@@ -153,6 +153,17 @@ class Norm(Part):
     returns the normed rows in the runtime's dtype."""
 
     def forward(self, x, delta=None, rows=None, write_x=True, delta_scale=1.0):
+        raise NotImplementedError
+
+
+class Side(Part):
+    """A part that joins something of its own to the stream behind a layer's sublayers:
+    ``forward(x, rows, ctx, mult, next_norm=None)``: x += mult * (what the part makes of `rows`), with `x`
+    the float32 stream and `rows` the same rows as a product's operand (the runtime's type).  With
+    `next_norm` (the norm that reads the stream next) the part may make that norm's rows in the kernel
+    that joins, and returns them; else None."""
+
+    def forward(self, x, rows, ctx, mult, next_norm=None):
         raise NotImplementedError
 
 

@@ -16,8 +16,8 @@ has the mixer sublayer only.  Such blocks take the plain path below (no deferred
 accumulation into the stream by the products).
 
 ``post_norm`` (further down) puts the norms on the sublayers' outputs instead, ``sandwich_norm`` on both
-sides of each sublayer, and ``sum_norm`` (at the end of this file) behind the residual sums, so that the
-normed rows are the stream.
+sides of each sublayer, ``sum_norm`` behind the residual sums, so that the normed rows are the stream, and
+``shared_norm`` (at the end of this file) has one norm whose rows both sublayers read.
 
 A block's interface: ``__init__(layer_spec, runtime)`` builds its parts from the registries;
 ``parts()`` lists them; ``forward(x, pending, ctx, cache) -> pending``.
@@ -286,3 +286,62 @@ class SumNormBlock:
             f = self.ffn.forward(h, ctx)
             self.norm_ffn.sum_norm(x, f, self.alpha, copy)
         return None
+
+
+@register_part("block", "shared_norm")
+class SharedNormBlock:
+    """One norm, both sublayers side by side behind it:
+
+        h = norm_mixer(x);  x += m * (mixer(h) + ffn(h));  then, with a `side` part, x += m * side(x)
+
+    with m the block parameter `residual_mult` (default 1); a spec without a feed-forward has the mixer alone.
+    The stream is float32.  A mixer that offers ``join`` (parts/parallel.py) adds its output and the
+    feed-forward's to the stream in the kernel that makes its output; the same kernel writes the rounded copy
+    of the stream that the side part's product reads.  The side part's last kernel may also make the rows of the
+    norm that the next block begins with (handed on as `PreparedRows`).  Nothing is owed to the stream when
+    the block returns."""
+
+    CAPTURE_SAFE = True
+    TRACEABLE = False
+    DEFERS_NORM = True            # the model hands `next_entry` to blocks that say so
+
+    def __init__(self, layer_spec, runtime):
+        self.runtime = runtime
+        self.mult = float(dict(getattr(layer_spec, "block_params", None) or {}).get("residual_mult", 1.0))
+        self.norm_mixer = build_part("norm", layer_spec.norms["mixer"], runtime)
+        self.mixer = build_part("mixer", layer_spec.mixer, runtime)
+        self.ffn = build_part("ffn", layer_spec.ffn, runtime) if layer_spec.ffn is not None else None
+        self.side = build_part("side", layer_spec.side, runtime) if layer_spec.side is not None else None
+        self.position = (build_part("position", layer_spec.position, runtime)
+                         if layer_spec.position is not None else None)
+        self.CAPTURE_SAFE = all(getattr(p, "CAPTURE_SAFE", False) for p in self.parts())
+
+    def parts(self):
+        return [p for p in (self.norm_mixer, self.mixer, self.ffn, self.side, self.position) if p is not None]
+
+    def entry(self):
+        return self.norm_mixer, self.mixer
+
+    def forward(self, x, pending, ctx, cache, next_entry=None):
+        import torch
+        if isinstance(pending, PreparedRows):
+            h = pending.h
+        elif pending is not None:
+            raise ValueError("shared_norm: the block before still owes the stream something; "
+                             "blocks of this kind join their outputs themselves")
+        else:
+            h = self.norm_mixer.forward(x)
+        f = self.ffn.forward(h, ctx) if self.ffn is not None else None
+        copy = None
+        if self.side is not None and not self.runtime.is_f32:
+            copy = torch.empty(x.shape, dtype=self.runtime.dtype, device=x.device)
+        if hasattr(self.mixer, "join"):
+            self.mixer.join(h, ctx, cache, self.position, x, f, self.mult, copy)
+        else:
+            a = self.mixer.forward(h, ctx, cache, self.position)
+            ops.join_sum_rows(a, x, self.mult, c=f, low=copy)
+        if self.side is None:
+            return None
+        rows = self.side.forward(x, x if copy is None else copy, ctx, self.mult,
+                                 next_entry[0] if next_entry is not None else None)
+        return PreparedRows(rows) if rows is not None else None

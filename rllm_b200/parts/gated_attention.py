@@ -14,8 +14,10 @@ For normed input rows h [n, d] (H query heads, G key/value heads, key size dk, v
                                                       `gate_per_head` Wg has one row per head and its
                                                       number multiplies the whole head)
 
+With `tie_values` there is no Wv: the values are the key rows as projected, before their norm.
+
 Parameters: hidden_size, num_heads, num_kv_heads, head_dim, v_head_dim, bias, qk_norm ("row" or
-None), eps, window (0: all keys), keep_first, scale, gate ("sigmoid" or None), gate_per_head.  Tensors under
+None), eps, window (0: all keys), keep_first, scale, gate ("sigmoid" or None), gate_per_head, tie_values.  Tensors under
 <prefix>: q, k, v, o, g and, by the options, q.b, k.b, v.b, q.norm, k.norm.  Load-time transform:
 q, k, v and the gate are stacked into one projection [q | k | v | g] (the biases of q, k, v likewise; rows of
 zeros up to a multiple of 8 rows).  Scores, softmax, norms and the
@@ -32,6 +34,7 @@ from .base import Mixer, PagedKVNeed, PartError, register_part
 @register_part("mixer", "gated_attention")
 class GatedWindowAttention(Mixer):
     CAPTURE_SAFE = True
+    INPUT_MATRIX = "w_qkv"        # the stacked product on h; a mixer made of mixers may run it with its neighbour's
 
     def __init__(self, params, prefix, runtime):
         super().__init__(params, prefix, runtime)
@@ -48,6 +51,9 @@ class GatedWindowAttention(Mixer):
         self.scale = float(p["scale"])
         self.gate = p.get("gate")
         self.gate_per_head = bool(p.get("gate_per_head", False)) and bool(self.gate)
+        self.tie_values = bool(p.get("tie_values", False))
+        if self.tie_values and (self.dv != self.dk or self.bias):
+            raise PartError("gated_attention: tied values have the keys' head size and no biases")
         if self.H % self.G:
             raise PartError(f"gated_attention: {self.H} heads are not a multiple of {self.G} key/value heads")
         if self.qk_norm not in (None, "row"):
@@ -64,8 +70,9 @@ class GatedWindowAttention(Mixer):
     def expected_tensors(self):
         d, p = self.hidden_size, self.prefix
         wq, wk, wv = self.H * self.dk, self.G * self.dk, self.G * self.dv
-        t = {p + "q": ((wq, d), "matrix"), p + "k": ((wk, d), "matrix"), p + "v": ((wv, d), "matrix"),
-             p + "o": ((d, self.H * self.dv), "matrix")}
+        t = {p + "q": ((wq, d), "matrix"), p + "k": ((wk, d), "matrix"), p + "o": ((d, self.H * self.dv), "matrix")}
+        if not self.tie_values:
+            t[p + "v"] = ((wv, d), "matrix")
         if self.bias:
             t.update({p + "q.b": ((wq,), "bias"), p + "k.b": ((wk,), "bias"), p + "v.b": ((wv,), "bias")})
         if self.qk_norm:
@@ -76,7 +83,7 @@ class GatedWindowAttention(Mixer):
 
     def load(self, tensors):
         p, dt = self.prefix, self.runtime.dtype
-        names = "qkvg" if self.gate else "qkv"
+        names = ("qk" if self.tie_values else "qkv") + ("g" if self.gate else "")
         stack = [tensors[p + n].to(dt) for n in names]
         rows = sum(t.shape[0] for t in stack)
         if rows % 8:                 # the projection's float32 rows stay aligned for every product kernel
@@ -90,10 +97,11 @@ class GatedWindowAttention(Mixer):
             self.k_norm_w = self._to_device(tensors[p + "k.norm"], torch.float32)
         self.w_o = self._to_device(tensors[p + "o"])
 
-    def forward(self, h, ctx, cache, position=None, residual=None):
+    def forward(self, h, ctx, cache, position=None, residual=None, rows=None):
+        """`rows`: h . w_qkv^T (float32), where somebody else has run that product."""
         n, dt, dev = h.shape[0], self.runtime.dtype, h.device
-        wide = ops.linear(h, self.w_qkv, out_dtype=torch.float32)          # [q | k | v | gate]
-        n_qkv = self.H * self.dk + self.G * (self.dk + self.dv)
+        wide = ops.linear(h, self.w_qkv, out_dtype=torch.float32) if rows is None else rows     # [q | k | v | gate]
+        n_qkv = (self.H + self.G) * self.dk + (0 if self.tie_values else self.G * self.dv)
         qkv = wide[:, :n_qkv]
         q = torch.empty((n, self.H * self.dk), dtype=dt, device=dev)
         rot = min(position.dims, self.dk) if position is not None else 0
@@ -102,7 +110,7 @@ class GatedWindowAttention(Mixer):
         ops.qkv_rownorm_store(qkv, self.b_qkv, self.q_norm_w, self.k_norm_w, cache.slots, q, cache.k, cache.v,
                               self.H, self.G, self.dk, self.dv, cache.block_size, self.eps, write_kv=cache.write,
                               cs_table=position.angles(ctx) if rot else None, rot=rot,
-                              pairs=bool(rot) and position.layout == "pairs")
+                              pairs=bool(rot) and position.layout == "pairs", v_tied=self.tie_values)
         attn = torch.empty((n, self.H * self.dv), dtype=dt, device=dev)
         ops.paged_attention(q, cache.k, cache.v, attn, ctx, cache.block_table, self.H, self.G, self.dk,
                             cache.block_size, self.scale, self.window, self.keep_first, self.dv)

@@ -11,13 +11,15 @@ For normed input rows h [n, d], E experts of size F, each token using `top_k`:
         minus infinity)
     the `top_k` experts with the largest c are chosen;  their weights are their s (without the
         correction), divided by their sum + `weight_eps` when `normalize`, times `route_scale`
-    expert e:  y_e = Wd_e (silu(Wg_e h) * (Wu_e h))
+    expert e:  y_e = Wd_e (silu(Wg_e h) * (Wu_e h)), or with `expert_form` = {limit, alpha, shift} the gated unit
+               Wd_e (g sigmoid(alpha g) (u + shift)), g = min(Wg_e h, limit), u = clamp(Wu_e h, -limit, limit)
     out = sum over the chosen e of weight_e * y_e
           + sigmoid(h . w_sg) * shared(h)                (`shared_size` > 0: one more expert of that size
-                                                          for every token; `shared_gate`: its gate)
+                                                          for every token; `shared_gate`: its gate;
+                                                          `shared_form`: its gated form, as above)
 
 Parameters: hidden_size, intermediate_size, num_experts, top_k, n_groups, keep_groups, group_best, score,
-correction, normalize, weight_eps, route_scale, shared_size, shared_gate, router_bias.  Tensors under <prefix>:
+correction, normalize, weight_eps, route_scale, shared_size, shared_gate, router_bias, expert_form, shared_form.  Tensors under <prefix>:
 router [E, d], router.b [E], correction [E], e<i>.gate, e<i>.up [F, d], e<i>.down [d, F], shared.gate, shared.up,
 shared.down, shared.sg [1, d].  Load-time transform: the experts' matrices are stacked ([E, 2F, d] gate
 rows then up rows, [E, d, F]), and the shared expert's gate row is stacked under the router's so that
@@ -58,6 +60,10 @@ class RoutedExperts(FeedForward):
         self.route_scale = float(p.get("route_scale", 1.0))
         self.shared_size = int(p.get("shared_size", 0) or 0)
         self.shared_gate = bool(p.get("shared_gate", False)) and self.shared_size > 0
+        form = lambda f: (float(f["limit"]), float(f["alpha"]), float(f["shift"])) if f else None
+        self.expert_form, self.shared_form = form(p.get("expert_form")), form(p.get("shared_form"))
+        if any(f is not None and f[1] == 0.0 for f in (self.expert_form, self.shared_form)):
+            raise PartError("routed_experts: a gated form's alpha must not be 0")
         if self.E % self.n_groups or not 0 < self.keep_groups <= self.n_groups:
             raise PartError(f"routed_experts: {self.E} experts do not form {self.n_groups} equal groups "
                             f"of which {self.keep_groups} are kept")
@@ -121,13 +127,13 @@ class RoutedExperts(FeedForward):
         shared = gate = None
         if self.shared_size:
             act = torch.empty((n, self.shared_size), dtype=dt, device=dev)
-            ops.gate_up_swiglu(h, self.w_shared_gu, act)
+            ops.gate_up_swiglu(h, self.w_shared_gu, act, glu=self.shared_form)
             shared = ops.linear(act, self.w_shared_down, out_dtype=torch.float32)
             gate = logits[:, self.E:self.E + 1] if self.shared_gate else None
         out = torch.empty((n, d), dtype=torch.float32, device=dev)
         if n <= PAIR_ROWS or torch.cuda.is_current_stream_capturing():
             act = torch.empty((n * self.top_k, self.F), dtype=dt, device=dev)
-            ops.moe_pairs_gate_up(h, self.w_gu, idx, act)
+            ops.moe_pairs_gate_up(h, self.w_gu, idx, act, glu=self.expert_form or (0.0, 1.0, 0.0))
             return ops.moe_pairs_down(act, self.w_down, idx, weight, out, shared, gate)
         # many rows: the pairs in expert order, each expert's rows through the package's products
         offsets, place = ops.moe_sort(idx, self.E)
@@ -139,6 +145,6 @@ class RoutedExperts(FeedForward):
         for e in range(self.E):
             a, b = bounds[e], bounds[e + 1]
             if b > a:
-                ops.gate_up_swiglu(rows[a:b], self.w_gu[e], act[a:b])
+                ops.gate_up_swiglu(rows[a:b], self.w_gu[e], act[a:b], glu=self.expert_form)
                 ops.linear(act[a:b], self.w_down[e], out=y[a:b])
         return ops.moe_combine(y, place, weight, out, shared, gate)

@@ -1,10 +1,18 @@
-"""Two mixers side by side on the same input: out = left_scale * left(h) + right_scale * right(h).
+"""Two mixers side by side on the same input: out = left_scale * left(h) + right_scale * right(h), each
+side's output optionally behind an RMS norm of its own (`left_norm`, `right_norm`: PartSpecs of norms).
 
 Parameters: left, right (PartSpec of registered mixer kinds, with their own prefixes), left_scale,
-right_scale.  Each side keeps what it needs in the cache under its own need; this part's need is
-the tuple of both and its cache view the tuple of their views.
+right_scale, left_norm, right_norm.  Each side keeps what it needs in the cache under its own need; this part's
+need is the tuple of both and its cache view the tuple of their views.
+
+Where both sides begin with one product on h (they name its matrix: INPUT_MATRIX), the two matrices are
+stacked at load and run as one product.  ``join(h, ctx, cache, position, x, extra, mult, copy)``: the kernel that
+norms and adds the two sides also adds `extra` (a feed-forward's output, or None) and joins the sum, times
+mult, to the float32 stream x; `copy`, if given, takes the new x in its own type.
 """
 from __future__ import annotations
+
+import torch
 
 from ..csrc import ops
 from .base import Mixer, build_part, register_part
@@ -17,19 +25,47 @@ class ParallelMixer(Mixer):
         self.left = build_part("mixer", params["left"], runtime)
         self.right = build_part("mixer", params["right"], runtime)
         self.left_scale, self.right_scale = float(params["left_scale"]), float(params["right_scale"])
+        norm = lambda key: build_part("norm", params[key], runtime) if params.get(key) else None
+        self.left_norm, self.right_norm = norm("left_norm"), norm("right_norm")
+        self.w_both = None
         self.CAPTURE_SAFE = bool(getattr(self.left, "CAPTURE_SAFE", False) and getattr(self.right, "CAPTURE_SAFE", False))
+
+    def _parts(self):
+        return [p for p in (self.left, self.right, self.left_norm, self.right_norm) if p is not None]
 
     def cache_need(self):
         return (self.left.cache_need(), self.right.cache_need())
 
     def expected_tensors(self):
-        return {**self.left.expected_tensors(), **self.right.expected_tensors()}
+        return {k: v for p in self._parts() for k, v in p.expected_tensors().items()}
 
     def load(self, tensors):
-        self.left.load(tensors)
-        self.right.load(tensors)
+        for p in self._parts():
+            p.load(tensors)
+        names = [getattr(s, "INPUT_MATRIX", None) for s in (self.left, self.right)]
+        if all(names):
+            ws = [getattr(s, n) for s, n in zip((self.left, self.right), names)]
+            self.w_both = torch.cat(ws, 0)
+            self.split = ws[0].shape[0]
+            setattr(self.left, names[0], self.w_both[:self.split])        # the sides keep views, not copies
+            setattr(self.right, names[1], self.w_both[self.split:])
+
+    def _sides(self, h, ctx, cache, position):
+        if self.w_both is None:
+            return (self.left.forward(h, ctx, cache[0], position), self.right.forward(h, ctx, cache[1], position))
+        rows = ops.linear(h, self.w_both, out_dtype=torch.float32)
+        return (self.left.forward(h, ctx, cache[0], position, rows=rows[:, :self.split]),
+                self.right.forward(h, ctx, cache[1], position, rows=rows[:, self.split:]))
+
+    def join(self, h, ctx, cache, position, x, extra=None, mult=1.0, copy=None, add=True):
+        a, b = self._sides(h, ctx, cache, position)
+        form = lambda n: (n.weight, n.eps) if n is not None else None
+        return ops.join_sum_rows(a, x, mult, add, form(self.left_norm), self.left_scale, b, form(self.right_norm),
+                                 self.right_scale, extra, copy)
 
     def forward(self, h, ctx, cache, position=None, residual=None):
-        a = self.left.forward(h, ctx, cache[0], position)
-        b = self.right.forward(h, ctx, cache[1], position)
-        return ops.axpby(self.left_scale, a, self.right_scale, b, a)
+        if self.left_norm is None and self.right_norm is None:
+            a, b = self._sides(h, ctx, cache, position)
+            return ops.axpby(self.left_scale, a, self.right_scale, b, a)
+        out = torch.empty(h.shape, dtype=torch.float32, device=h.device)
+        return self.join(h, ctx, cache, position, out, add=False)
