@@ -196,9 +196,26 @@ def navulorn_shape(width: int) -> dict:
             "logit_softcap": 30.0}
 
 
-FAMILY_SHAPES = {"falalix": falalix_shape, "govopel": govopel_shape, "divuzen": divuzen_shape, "navulorn": navulorn_shape}
+def rusolorn_shape(width: int) -> dict:
+    """A Rusolorn configuration with layer sizes of a real model of that width: six layers, each with windowed
+    attention (width/128 heads of 128, a quarter as many key/value heads, a window of 1,024 keys) beside the gated
+    delta rule (width/128 value heads of 128 on half as many query/key heads of 128, convolutions of 4 taps), 16
+    clamped experts of 3/8 width of which a token uses 4, in 4 groups of which 2 are kept, a shared one of 3/4 width,
+    and a token input of 256 entries."""
+    heads = max(8, width // 128)
+    left = {"heads": heads, "kv_heads": max(1, heads // 4), "dim": 128, "vdim": 128, "mask": {"size": 1024}, "scale": 128 ** -0.5}
+    right = {"heads": heads, "kv_heads": heads // 2, "dim": 128, "vdim": 128, "conv": 4}
+    moe = {"kind": "moe", "expert": {"ff": 3 * width // 8, "limit": 7.0}, "shared": {"ff": 3 * width // 4, "limit": 7.0},
+           "router": {"experts": 16, "top": 4, "groups": {"count": 4, "keep": 2}}}
+    layer = {"type": "parallel", "mixer": {"left": left, "right": right}, "mlp": moe}
+    return {"architecture": "Rusolorn", "vocab": 32768, "width": width, "layers": [layer] * 6, "norm": {"eps": 1e-6},
+            "embedding": {"scale": 8.0}, "residual_mult": 0.5, "token_side": {"dim": 256}}
+
+
+FAMILY_SHAPES = {"falalix": falalix_shape, "govopel": govopel_shape, "divuzen": divuzen_shape, "navulorn": navulorn_shape,
+                 "rusolorn": rusolorn_shape}
 # the model a family stands beside: Qwen3-shaped of equal width, depth and feed-forward, unless another family is closer
-BESIDE = {"navulorn": "divuzen"}
+BESIDE = {"navulorn": "divuzen", "rusolorn": "divuzen"}
 
 
 def falalix_compare(a):
@@ -216,7 +233,7 @@ def falalix_compare(a):
     widths = {"1k": 1024, "2k": 2048, "4k": 4096}
     family = a.workload
     other = BESIDE.get(family, "qwen3")
-    out = {"metric": f"{family.capitalize()}-shaped against {other.capitalize()}-shaped models of equal width and depth: prefill tok/s "
+    out = {"metric": f"{family.capitalize()}-shaped against {other.capitalize()}-shaped models of equal width: prefill tok/s "
                      "(2,048 tokens, one step) and decode tok/s (batch 8, 2,048-token prompts)",
            "unit": "tok/s", "n_gpus": 1, "steps": a.steps, "warmup": a.warmup, "dtype": "bf16", "impl": "ours",
            "data": "synthetic: random weights, uniform random token ids", "sizes": {}}
@@ -311,14 +328,15 @@ def main():
     ap.add_argument("--ctx", type=int, default=None, help="tokens a request may hold (default: twice the prompt)")
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--skip-points", action="store_true", help="leave out batch 1 / 64 and prefill")
-    ap.add_argument("--workload", default="decode", choices=["decode", "serving", "falalix", "govopel", "divuzen", "navulorn"],
+    ap.add_argument("--workload", default="decode", choices=["decode", "serving", "falalix", "govopel", "divuzen", "navulorn", "rusolorn"],
                     help="decode: the default line.  serving: --requests prompts of 16..2,048 tokens with 128..512 "
                          "generated tokens each through LLM.generate (continuous batching), one line of its own.  "
                          "falalix: prefill and decode of Falalix-shaped models (--sizes) beside Qwen3-shaped models of "
                          "equal width, depth and feed-forward, one line of its own.  govopel, divuzen: the same for "
                          "Govopel-shaped and for Divuzen-shaped models.  navulorn: Navulorn-shaped beside Divuzen-shaped "
-                         "models of equal width and depth")
-    ap.add_argument("--sizes", default="1k,2k,4k", help="falalix, govopel, divuzen, navulorn: model widths to run (1k, 2k, 4k)")
+                         "models of equal width and depth.  rusolorn: Rusolorn-shaped beside Divuzen-shaped models "
+                         "of equal width and about equal weights (six layers of two mixers each beside eight of one)")
+    ap.add_argument("--sizes", default="1k,2k,4k", help="falalix, govopel, divuzen, navulorn, rusolorn: model widths to run (1k, 2k, 4k)")
     ap.add_argument("--requests", type=int, default=64)
     ap.add_argument("--parallel", type=int, default=32, help="serving: requests running at once")
     ap.add_argument("--prefill-chunk", type=int, default=512, help="serving: prompt tokens per step")

@@ -21,10 +21,10 @@
 //   delta_step    (few tokens per request: decode) one block per (head, request) does all of the above, the
 //                 recurrence token by token with S in registers.
 //   delta_prep, delta_chunk, delta_out  (prompt portions) chunks of 8 tokens, counted from the portion's start.
-//                 prep: a block per (chunk, q/k head): convolutions and unit vectors of q and k, the products
-//                 k_i . k_j and q_i . k_j inside the chunk, beta and g.  chunk: a block per (tile of value
-//                 columns, head, request) walks the request's chunks with its part of S in registers.  With
-//                 c_i = g_1 .. g_i and d_ij = g_(j+1) .. g_i (products taken factor by factor, from 1):
+//                 prep: a block per (chunk, q/k head): convolutions and unit vectors of q and k, and the small
+//                 matrices below.  chunk: a block per (tile of value columns, head, request) walks the
+//                 request's chunks with its part of S in registers.  With c_i = g_1 .. g_i and d_ij =
+//                 g_(j+1) .. g_i (products taken factor by factor, never as a quotient):
 //                     u_i = beta_i (v_i - c_i S0^T k_i) - sum_(j<i) beta_i d_ij (k_i . k_j) u_j
 //                     o_i = c_i S0^T q_i + sum_(j<=i) d_ij (q_i . k_j) u_j
 //                     S   = c_8 S0 + sum_j d_8j k_j u_j^T
@@ -86,8 +86,10 @@ __device__ __forceinline__ void head_channel(const DeltaArgs& p, int h, int c, i
 }
 
 // ------------------------------------------------------------------ few tokens: one block per (head, request)
+constexpr int delta_step_threads(int DK) { return DK > 256 ? 256 : 512; }
+
 template <typename TA, int DK>
-__global__ void __launch_bounds__(512)
+__global__ void __launch_bounds__(delta_step_threads(DK), DK <= 128 ? 2 : 1)
 delta_step_kernel(const DeltaArgs p, TA* out) {
     constexpr int IPT = DK / DELTA_PARTS;
     extern __shared__ __align__(16) float sm_step[];
@@ -237,14 +239,34 @@ delta_step_kernel(const DeltaArgs p, TA* out) {
 }
 
 // ------------------------------------------------------------------ portions: what a chunk needs beside the memory
-// qn, kn [n, G * dk]: the unit vectors (q times q_scale).  prods [n, G, 16]: token i of a chunk has k_i . k_j at
-// [j] and q_i . k_j at [8 + j] for j <= i.  bg [n, H, 2]: beta and g.
+// Chunks are numbered through the step's requests in order.  qn, kn [n, G * dk]: the unit vectors (q times
+// q_scale).  mats [chunks, H, DELTA_MAT]: -beta_i d_ij (k_i . k_j) at [8 i + j], every entry twice (a pair that
+// multiplies two columns at once); d_ij (q_i . k_j) at [128 + 8 i + j] (0 for j > i); beta_i, c_i, d_8i at [192 + i], [200 + i],
+// [208 + i].  Tokens behind the last one of a short chunk have k = q = 0, beta = 0 and g = 1.
+#define DELTA_MAT 216
+
+// Sixteen values summed over a warp; lane l ends with the sum of value number l / 2.
+__device__ __forceinline__ float reduce16(const float (&a)[16], int lane) {
+    float b[8], c[4], d[2];
+    const bool h4 = lane & 16, h3 = lane & 8, h2 = lane & 4, h1 = lane & 2;
+#pragma unroll
+    for (int j = 0; j < 8; ++j) b[j] = (h4 ? a[8 + j] : a[j]) + __shfl_xor_sync(0xffffffffu, h4 ? a[j] : a[8 + j], 16);
+#pragma unroll
+    for (int j = 0; j < 4; ++j) c[j] = (h3 ? b[4 + j] : b[j]) + __shfl_xor_sync(0xffffffffu, h3 ? b[j] : b[4 + j], 8);
+#pragma unroll
+    for (int j = 0; j < 2; ++j) d[j] = (h2 ? c[2 + j] : c[j]) + __shfl_xor_sync(0xffffffffu, h2 ? c[j] : c[2 + j], 4);
+    const float e = (h1 ? d[1] : d[0]) + __shfl_xor_sync(0xffffffffu, h1 ? d[0] : d[1], 2);
+    return e + __shfl_xor_sync(0xffffffffu, e, 1);
+}
+
 __global__ void __launch_bounds__(256)
-delta_prep_kernel(const DeltaArgs p, float* qn, float* kn, float* prods, float* bg) {
+delta_prep_kernel(const DeltaArgs p, float* qn, float* kn, float* mats) {
     extern __shared__ __align__(16) float sm_prep[];
     float* s_q = sm_prep;                            // [TOK][dk]
     float* s_k = s_q + DELTA_TOK * p.dk;
-    pdl_launch_dependents();
+    float* s_bg = s_k + DELTA_TOK * p.dk;            // [rep][2][TOK]: beta, g
+    __shared__ float s_pr[DELTA_TOK][2 * DELTA_TOK]; // k_i . k_j, q_i . k_j
+    // (no early launch of what follows: the chunk kernel's few, long-lived blocks are to spread over idle SMs)
     pdl_wait();
     int chunk = blockIdx.x, r = 0, len = 0;
     for (; r < p.n_requests; ++r) {
@@ -259,6 +281,17 @@ delta_prep_kernel(const DeltaArgs p, float* qn, float* kn, float* prods, float* 
     const float* x0 = p.rows + (size_t)t0 * p.ld;
     const int C = 2 * p.dk + p.dv;
     const float* kept = p.state + (size_t)p.slots[r] * p.slot_stride + p.conv_base + (size_t)kh * rep * C * (p.taps - 1);
+    for (int e = tid; e < DELTA_TOK * rep; e += blockDim.x) {
+        const int i = e & 7, hh = e >> 3, h = kh * rep + hh;
+        float beta = 0.f, g = 1.f;
+        if (i < cnt) {
+            const float* row = x0 + (size_t)(c0 + i) * p.ld;
+            beta = 1.0f / (1.0f + expf(-row[p.b_off + h]));
+            g = head_decay(p, h, row[p.a_off + h]);
+        }
+        s_bg[hh * 2 * DELTA_TOK + i] = beta;
+        s_bg[hh * 2 * DELTA_TOK + DELTA_TOK + i] = g;
+    }
     for (int c = tid; c < 2 * p.dk; c += blockDim.x) {       // a thread takes a channel's tokens
         const bool is_k = c >= p.dk;
         const int cc = is_k ? c - p.dk : c;
@@ -282,7 +315,8 @@ delta_prep_kernel(const DeltaArgs p, float* qn, float* kn, float* prods, float* 
         }
     }
     __syncthreads();
-    for (int i = warp; i < cnt; i += 8) {
+    if (warp < cnt) {                                // warp i: token i's lengths
+        const int i = warp;
         float qq = 0.f, kk = 0.f;
         for (int c = lane; c < p.dk; c += 32) {
             qq += s_q[i * p.dk + c] * s_q[i * p.dk + c];
@@ -297,32 +331,40 @@ delta_prep_kernel(const DeltaArgs p, float* qn, float* kn, float* prods, float* 
         }
     }
     __syncthreads();
-    for (int i = warp; i < cnt; i += 8) {
-        float kk[DELTA_TOK], qk[DELTA_TOK];
+    {                                                // and its products with the keys up to it
+        const int i = warp;
+        float pr[16];
 #pragma unroll
-        for (int j = 0; j < DELTA_TOK; ++j) kk[j] = qk[j] = 0.f;
-        for (int c = lane; c < p.dk; c += 32) {
-            const float a = s_q[i * p.dk + c], b = s_k[i * p.dk + c];
+        for (int j = 0; j < 16; ++j) pr[j] = 0.f;
+        if (i < cnt)
+            for (int c = lane; c < p.dk; c += 32) {
+                const float a = s_q[i * p.dk + c], b = s_k[i * p.dk + c];
 #pragma unroll
-            for (int j = 0; j < DELTA_TOK; ++j) {
-                const float o = j <= i ? s_k[j * p.dk + c] : 0.f;
-                kk[j] += b * o;
-                qk[j] += a * o;
+                for (int j = 0; j < DELTA_TOK; ++j) {
+                    const float o = j <= i ? s_k[j * p.dk + c] : 0.f;
+                    pr[j] += b * o;
+                    pr[DELTA_TOK + j] += a * o;
+                }
             }
-        }
-        float* dst = prods + ((size_t)(t0 + c0 + i) * p.G + kh) * 2 * DELTA_TOK;
-#pragma unroll
-        for (int j = 0; j < DELTA_TOK; ++j) {
-            const float a = warp_sum(kk[j]), b = warp_sum(qk[j]);
-            if (lane == 0) { dst[j] = a; dst[DELTA_TOK + j] = b; }
-        }
+        const float v = reduce16(pr, lane);
+        if (!(lane & 1)) s_pr[i][lane >> 1] = v;
     }
-    for (int e = tid; e < cnt * rep; e += blockDim.x) {
-        const int i = e / rep, h = kh * rep + e % rep;
-        const size_t t = t0 + c0 + i;
-        const float* row = p.rows + t * p.ld;
-        bg[(t * p.H + h) * 2] = 1.0f / (1.0f + expf(-row[p.b_off + h]));
-        bg[(t * p.H + h) * 2 + 1] = head_decay(p, h, row[p.a_off + h]);
+    __syncthreads();
+    for (int e = tid; e < rep * 64; e += blockDim.x) {
+        const int hh = e >> 6, i = (e >> 3) & 7, j = e & 7;
+        const float *beta = s_bg + hh * 2 * DELTA_TOK, *g = beta + DELTA_TOK;
+        float d = 1.f;
+#pragma unroll
+        for (int m = 1; m < DELTA_TOK; ++m) d *= (m > j && m <= i) ? g[m] : 1.f;
+        float* dst = mats + ((size_t)blockIdx.x * p.H + kh * rep + hh) * DELTA_MAT;
+        const float kk = j < i ? -beta[i] * d * s_pr[i][j] : 0.f;
+        *reinterpret_cast<float2*>(dst + 2 * (8 * i + j)) = make_float2(kk, kk);
+        dst[128 + 8 * i + j] = j <= i ? d * s_pr[i][DELTA_TOK + j] : 0.f;
+        if (j == 0) {
+            dst[192 + i] = beta[i];
+            dst[200 + i] = d * g[0];
+        }
+        if (i == DELTA_TOK - 1) dst[208 + j] = d;
     }
 }
 
@@ -333,10 +375,37 @@ __device__ __forceinline__ void delta_cp4(float* dst, const float* src) {
 __device__ __forceinline__ void delta_cp16(float* dst, const float* src) {
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src));
 }
+// Pairs of floats in one 64-bit register: two multiply-adds an instruction (each rounded as a single one is).
+typedef unsigned long long f2;
+__device__ __forceinline__ f2 f2_make(float a, float b) {
+    f2 r;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b));
+    return r;
+}
+__device__ __forceinline__ void f2_split(f2 v, float& a, float& b) { asm("mov.b64 {%0, %1}, %2;" : "=f"(a), "=f"(b) : "l"(v)); }
+__device__ __forceinline__ f2 f2_fma(f2 a, f2 b, f2 c) {
+    f2 r;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+    return r;
+}
+__device__ __forceinline__ f2 f2_mul(f2 a, f2 b) {
+    f2 r;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+    return r;
+}
+// Keeps the compiler from requesting the operands of later work here: they would not fit the registers.
+__device__ __forceinline__ void hold_loads() { asm volatile("" ::: "memory"); }
+__device__ __forceinline__ float f2_sum(f2 v) {
+    float a, b;
+    f2_split(v, a, b);
+    return a + b;
+}
 // Sums of eight values over the eight lanes of a group; lane `part` ends with the sum of value number `part`.
-__device__ __forceinline__ float reduce8(const float (&a)[DELTA_TOK], int part) {
-    float b[4], c[2];
+__device__ __forceinline__ float reduce8(const f2 (&v)[DELTA_TOK], int part) {
+    float a[8], b[4], c[2];
     const bool h4 = part & 4, h2 = part & 2, h1 = part & 1;
+#pragma unroll
+    for (int j = 0; j < 8; ++j) a[j] = f2_sum(v[j]);
 #pragma unroll
     for (int j = 0; j < 4; ++j) b[j] = (h4 ? a[4 + j] : a[j]) + __shfl_xor_sync(0xffffffffu, h4 ? a[j] : a[4 + j], 4);
 #pragma unroll
@@ -349,15 +418,11 @@ __device__ __forceinline__ float reduce8(const float (&a)[DELTA_TOK], int part) 
 
 template <int DK>
 __global__ void __launch_bounds__(DELTA_NT)
-delta_chunk_kernel(const DeltaArgs p, const float* qn, const float* kn, const float* prods, const float* bg, float* o) {
-    constexpr int IPT = DK / DELTA_PARTS, T = DELTA_TOK, NC = DELTA_COLS;
+delta_chunk_kernel(const DeltaArgs p, const float* qn, const float* kn, const float* mats, float* o) {
+    constexpr int IPT = DK / DELTA_PARTS, T = DELTA_TOK, NC = DELTA_COLS, ROW4 = DK / 4;
     extern __shared__ __align__(16) float sm_chunk[];
     const int W = T + p.taps - 1;                    // rows of the values' window
-    const int stage = 2 * T * DK + T * 16 + 2 * T + (W * NC + 3) / 4 * 4;
-    float* s_kk = sm_chunk + 2 * stage;              // [T][T] beta_i d_ij (k_i . k_j), j < i
-    float* s_qk = s_kk + T * T;                      // [T][T] d_ij (q_i . k_j), j <= i, else 0
-    float* s_c = s_qk + T * T;                       // [T] c_i
-    float* s_d = s_c + T;                            // [T] d_8j
+    const int stage = 2 * T * DK + DELTA_MAT + W * NC;
     const int tid = threadIdx.x, part = tid & 7, lane = tid & 31;
     const int n_tiles = (p.dvp + NC - 1) / NC, h = blockIdx.x / n_tiles, tile = blockIdx.x % n_tiles, r = blockIdx.y;
     const int kh = h / (p.H / p.G), C = 2 * p.dk + p.dv;
@@ -365,6 +430,8 @@ delta_chunk_kernel(const DeltaArgs p, const float* qn, const float* kn, const fl
     pdl_wait();
     const int t0 = p.cu_q[r], len = p.cu_q[r + 1] - t0;
     if (len <= 0) return;
+    int chunk0 = 0;                                  // the number of the request's first chunk
+    for (int i = 0; i < r; ++i) chunk0 += (p.cu_q[i + 1] - p.cu_q[i] + T - 1) / T;
     float* slot = p.state + (size_t)p.slots[r] * p.slot_stride;
     float* Sg = slot + (size_t)h * DK * p.dvp;
     float* kept = slot + p.conv_base + (size_t)h * C * (p.taps - 1);
@@ -374,169 +441,184 @@ delta_chunk_kernel(const DeltaArgs p, const float* qn, const float* kn, const fl
     const bool live = 2 * pair < p.dvp;
     const size_t stride = (size_t)p.dvp * 4;
     const bool vec = (p.dk & 3) == 0;
-    float S0[IPT], S1[IPT];
+    f2 S0[IPT / 2], S1[IPT / 2];                     // rows ii, ii + 1 of the pair's two columns
 #pragma unroll
-    for (int ii = 0; ii < IPT; ++ii) {
-        S0[ii] = live ? Sg[(size_t)(2 * ii) * stride + gt] : 0.f;
-        S1[ii] = live ? Sg[(size_t)(2 * ii + 1) * stride + gt] : 0.f;
+    for (int m = 0; m < IPT / 2; ++m) {
+        const float* at = Sg + (size_t)(4 * m) * stride + gt;
+        S0[m] = live ? f2_make(at[0], at[2 * stride]) : 0ull;
+        S1[m] = live ? f2_make(at[stride], at[3 * stride]) : 0ull;
     }
-    // both stages start as zeros: the columns behind dk and behind the last token's rows are never filled
+    // both stages start as zeros: the columns behind dk and behind dv are never filled
     for (int e = tid; e < 2 * stage; e += DELTA_NT) sm_chunk[e] = 0.f;
     __syncthreads();
+    const float* v_src = x0 + p.v_off + (size_t)h * p.dv + col0;
+    const size_t tok_stride = (size_t)p.G * p.dk;
+    const float* mat_src = mats + ((size_t)chunk0 * p.H + h) * DELTA_MAT;
     auto fetch = [&](int c0, float* st) {
         const int cnt = min(T, len - c0);
-        float *q = st, *k = st + T * DK, *pr = k + T * DK, *b = pr + T * 16, *v = b + 2 * T;
-        const size_t t = t0 + c0;
+        float *q = st, *k = st + T * DK, *m = k + T * DK, *v = m + DELTA_MAT;
+        const size_t src = (size_t)(t0 + c0) * tok_stride + (size_t)kh * p.dk;
         if (vec) {
-            const int d4 = p.dk >> 2;
-            for (int e = tid; e < cnt * d4; e += DELTA_NT) {
-                const int i = e / d4, c = 4 * (e - i * d4);
-                const size_t src = ((t + i) * p.G + kh) * p.dk + c;
-                delta_cp16(q + i * DK + c, qn + src);
-                delta_cp16(k + i * DK + c, kn + src);
+#pragma unroll
+            for (int it = 0; it < (T * ROW4 + DELTA_NT - 1) / DELTA_NT; ++it) {
+                const int e = tid + it * DELTA_NT, i = e / ROW4, c = 4 * (e % ROW4);
+                if (i < cnt && c < p.dk) {
+                    delta_cp16(q + i * DK + c, qn + src + i * tok_stride + c);
+                    delta_cp16(k + i * DK + c, kn + src + i * tok_stride + c);
+                }
             }
         } else {
-            for (int e = tid; e < cnt * p.dk; e += DELTA_NT) {
-                const int i = e / p.dk, c = e - i * p.dk;
-                const size_t src = ((t + i) * p.G + kh) * p.dk + c;
-                delta_cp4(q + i * DK + c, qn + src);
-                delta_cp4(k + i * DK + c, kn + src);
+            for (int e = tid; e < cnt * DK; e += DELTA_NT) {
+                const int i = e / DK, c = e % DK;
+                if (c >= p.dk) continue;
+                delta_cp4(q + e, qn + src + i * tok_stride + c);
+                delta_cp4(k + e, kn + src + i * tok_stride + c);
             }
         }
-        if (tid < 4 * cnt) delta_cp16(pr + 4 * tid, prods + ((t + tid / 4) * p.G + kh) * 16 + 4 * (tid & 3));
-        if (tid < 2 * cnt) delta_cp4(b + tid, bg + ((t + tid / 2) * p.H + h) * 2 + (tid & 1));
-        for (int e = tid; e < (cnt + p.taps - 1) * NC; e += DELTA_NT) {
-            const int i = e / NC, c = col0 + e % NC;
-            if (c >= p.dv) continue;
-            const int s = c0 + i - (p.taps - 1);
-            delta_cp4(v + e, s >= 0 ? x0 + (size_t)s * p.ld + p.v_off + (size_t)h * p.dv + c
-                                    : kept_v + (size_t)c * (p.taps - 1) + p.taps - 1 + s);
-        }
+        if (tid < DELTA_MAT / 4) delta_cp16(m + 4 * tid, mat_src + (size_t)(c0 / T) * p.H * DELTA_MAT + 4 * tid);
+        const int c = tid % NC;
+        if (col0 + c < p.dv)
+            for (int i = tid / NC; i < cnt + p.taps - 1; i += DELTA_NT / NC) {
+                const int s = c0 + i - (p.taps - 1);
+                delta_cp4(v + i * NC + c, s >= 0 ? v_src + (size_t)s * p.ld + c
+                                                 : kept_v + (size_t)(col0 + c) * (p.taps - 1) + p.taps - 1 + s);
+            }
         asm volatile("cp.async.commit_group;\n" ::);
     };
     const float* wv0 = p.conv + (size_t)(2 * p.G * p.dk + h * p.dv + min(col0 + cl, p.dv - 1)) * p.taps;
     const float* wv1 = p.conv + (size_t)(2 * p.G * p.dk + h * p.dv + min(col0 + cl + 1, p.dv - 1)) * p.taps;
+    float w4a[4] = {0.f, 0.f, 0.f, 0.f}, w4b[4] = {0.f, 0.f, 0.f, 0.f};       // the usual four taps stay in registers
+    if (p.taps == 4)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) { w4a[j] = wv0[j]; w4b[j] = wv1[j]; }
+    float* dst = o + ((size_t)(t0 + part) * p.H + h) * p.dv + col0 + cl;
+    const bool st_a = col0 + cl < p.dv, st_b = col0 + cl + 1 < p.dv;
     fetch(0, sm_chunk);
     int buf = 0;
     for (int c0 = 0; c0 < len; c0 += T, buf ^= 1) {
         const int cnt = min(T, len - c0);
         float* st = sm_chunk + buf * stage;
         asm volatile("cp.async.wait_group 0;\n" ::);
-        __syncthreads();
-        float *s_q = st, *s_k = st + T * DK, *s_pr = s_k + T * DK, *s_b = s_pr + T * 16, *s_v = s_b + 2 * T;
+        __syncthreads();                             // this chunk is there, and everybody is done with the other stage
+        if (c0 + T < len) fetch(c0 + T, sm_chunk + (buf ^ 1) * stage);
+        float *s_q = st, *s_k = st + T * DK, *s_m = s_k + T * DK, *s_v = s_m + DELTA_MAT;
         if (cnt < T) {                               // the last, short chunk: rows that an earlier chunk left here are cleared
             for (int e = tid; e < (T - cnt) * DK; e += DELTA_NT) s_q[cnt * DK + e] = s_k[cnt * DK + e] = 0.f;
-            for (int e = tid; e < (T - cnt) * 16; e += DELTA_NT) s_pr[cnt * 16 + e] = 0.f;
-            if (tid < T - cnt) { s_b[2 * (cnt + tid)] = 0.f; s_b[2 * (cnt + tid) + 1] = 1.f; }
             __syncthreads();
         }
-        {                                            // thread (i, j) of 64 twice: the chunk's small matrices
-            const int e = tid & 63, i = e >> 3, j = e & 7;
-            float d = 1.f;
-            for (int m = j + 1; m <= i; ++m) d *= s_b[2 * m + 1];
-            if (tid < 64) {
-                s_kk[e] = j < i ? s_b[2 * i] * d * s_pr[i * 16 + j] : 0.f;
-                if (i == T - 1) s_d[j] = d;
-            } else {
-                s_qk[e] = j <= i ? d * s_pr[i * 16 + 8 + j] : 0.f;
-                if (j == 0) s_c[i] = d * s_b[1];
+        f2 ka[T], kb[T], qa[T], qb[T];
+#pragma unroll
+        for (int i = 0; i < T; ++i) ka[i] = kb[i] = qa[i] = qb[i] = 0ull;
+        // four tokens at a time: their operands first, then sixteen independent multiply-adds, then the other halves
+#pragma unroll
+        for (int m = 0; m < IPT / 4; ++m) {
+#pragma unroll
+            for (int i0 = 0; i0 < T; i0 += 4) {
+                ulonglong2 k[4], q[4];
+#pragma unroll
+                for (int i = 0; i < 4; ++i) {
+                    k[i] = *(reinterpret_cast<const ulonglong2*>(s_k + (i0 + i) * DK + 32 * m) + part);
+                    q[i] = *(reinterpret_cast<const ulonglong2*>(s_q + (i0 + i) * DK + 32 * m) + part);
+                }
+#pragma unroll
+                for (int i = 0; i < 4; ++i) {
+                    ka[i0 + i] = f2_fma(k[i].x, S0[2 * m], ka[i0 + i]);
+                    kb[i0 + i] = f2_fma(k[i].x, S1[2 * m], kb[i0 + i]);
+                    qa[i0 + i] = f2_fma(q[i].x, S0[2 * m], qa[i0 + i]);
+                    qb[i0 + i] = f2_fma(q[i].x, S1[2 * m], qb[i0 + i]);
+                }
+#pragma unroll
+                for (int i = 0; i < 4; ++i) {
+                    ka[i0 + i] = f2_fma(k[i].y, S0[2 * m + 1], ka[i0 + i]);
+                    kb[i0 + i] = f2_fma(k[i].y, S1[2 * m + 1], kb[i0 + i]);
+                    qa[i0 + i] = f2_fma(q[i].y, S0[2 * m + 1], qa[i0 + i]);
+                    qb[i0 + i] = f2_fma(q[i].y, S1[2 * m + 1], qb[i0 + i]);
+                }
             }
         }
         float va = 0.f, vb = 0.f;                    // this lane's token's values
-        for (int j = 0; j < p.taps; ++j) {
-            const float2 x = *reinterpret_cast<const float2*>(s_v + (part + j) * NC + cl);
-            va += wv0[j] * x.x;
-            vb += wv1[j] * x.y;
+        if (p.taps == 4) {
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+                const float2 x = *reinterpret_cast<const float2*>(s_v + (part + j) * NC + cl);
+                va += w4a[j] * x.x;
+                vb += w4b[j] * x.y;
+            }
+        } else {
+            for (int j = 0; j < p.taps; ++j) {
+                const float2 x = *reinterpret_cast<const float2*>(s_v + (part + j) * NC + cl);
+                va += wv0[j] * x.x;
+                vb += wv1[j] * x.y;
+            }
         }
         va = silu_f(va);
         vb = silu_f(vb);
-        float ka[T], kb[T], qa[T], qb[T];
-#pragma unroll
-        for (int i = 0; i < T; ++i) ka[i] = kb[i] = qa[i] = qb[i] = 0.f;
-#pragma unroll
-        for (int m = 0; m < IPT / 4; ++m) {
-#pragma unroll
-            for (int i = 0; i < T; ++i) {
-                const float4 k = *(reinterpret_cast<const float4*>(s_k + i * DK + 32 * m) + part);
-                ka[i] += k.x * S0[4 * m] + k.y * S0[4 * m + 1] + k.z * S0[4 * m + 2] + k.w * S0[4 * m + 3];
-                kb[i] += k.x * S1[4 * m] + k.y * S1[4 * m + 1] + k.z * S1[4 * m + 2] + k.w * S1[4 * m + 3];
-                const float4 q = *(reinterpret_cast<const float4*>(s_q + i * DK + 32 * m) + part);
-                qa[i] += q.x * S0[4 * m] + q.y * S0[4 * m + 1] + q.z * S0[4 * m + 2] + q.w * S0[4 * m + 3];
-                qb[i] += q.x * S1[4 * m] + q.y * S1[4 * m + 1] + q.z * S1[4 * m + 2] + q.w * S1[4 * m + 3];
-            }
-        }
         const float ksa = reduce8(ka, part), ksb = reduce8(kb, part), qsa = reduce8(qa, part), qsb = reduce8(qb, part);
-        __syncthreads();                             // the small matrices are there, and the other stage is free
-        if (c0 + T < len) fetch(c0 + T, sm_chunk + (buf ^ 1) * stage);
-        const float c = s_c[part], beta = s_b[2 * part];
+        const float beta = s_m[192 + part], c = s_m[200 + part];
         const float ra = beta * (va - c * ksa), rb = beta * (vb - c * ksb);
-        float ua[T], ub[T];
+        f2 u[T];                                     // the tokens' corrections of the two columns
 #pragma unroll
-        for (int i = 0; i < T; ++i) {
-            ua[i] = __shfl_sync(0xffffffffu, ra, (lane & 24) | i);
-            ub[i] = __shfl_sync(0xffffffffu, rb, (lane & 24) | i);
-        }
+        for (int i = 0; i < T; ++i)
+            u[i] = f2_make(__shfl_sync(0xffffffffu, ra, (lane & 24) | i), __shfl_sync(0xffffffffu, rb, (lane & 24) | i));
+        const f2* kk = reinterpret_cast<const f2*>(s_m);
 #pragma unroll
-        for (int i = 1; i < T; ++i)
+        for (int j = 0; j < T - 1; ++j)
 #pragma unroll
-            for (int j = 0; j < i; ++j) {
-                ua[i] -= s_kk[i * T + j] * ua[j];
-                ub[i] -= s_kk[i * T + j] * ub[j];
-            }
+            for (int i = j + 1; i < T; ++i) u[i] = f2_fma(kk[i * T + j], u[j], u[i]);
         float oa = c * qsa, ob = c * qsb;
 #pragma unroll
         for (int j = 0; j < T; ++j) {
-            const float w = s_qk[part * T + j];
-            oa += w * ua[j];
-            ob += w * ub[j];
+            const float w = s_m[128 + part * T + j];
+            float a, b;
+            f2_split(u[j], a, b);
+            oa += w * a;
+            ob += w * b;
         }
-        if (part < cnt && live) {
-            float* dst = o + ((size_t)(t0 + c0 + part) * p.H + h) * p.dv + col0 + cl;
-            if (col0 + cl < p.dv) dst[0] = oa;
-            if (col0 + cl + 1 < p.dv) dst[1] = ob;
+        if (part < cnt) {
+            if (st_a) dst[0] = oa;
+            if (st_b) dst[1] = ob;
         }
-        const float cT = s_c[T - 1];
+        dst += (size_t)T * p.H * p.dv;
+        const f2 cT = f2_make(s_m[200 + T - 1], s_m[200 + T - 1]);
+        f2 ua[T], ub[T];
 #pragma unroll
         for (int j = 0; j < T; ++j) {
-            const float w = s_d[j];
-            ua[j] *= w;
-            ub[j] *= w;
+            const float w = s_m[208 + j];
+            float a, b;
+            f2_split(u[j], a, b);
+            ua[j] = f2_make(a * w, a * w);
+            ub[j] = f2_make(b * w, b * w);
+        }
+        hold_loads();
+#pragma unroll
+        for (int m = 0; m < IPT / 2; ++m) {
+            S0[m] = f2_mul(S0[m], cT);
+            S1[m] = f2_mul(S1[m], cT);
         }
 #pragma unroll
-        for (int m = 0; m < IPT / 4; ++m) {
+        for (int j = 0; j < T; ++j)
 #pragma unroll
-            for (int e = 0; e < 4; ++e) {
-                S0[4 * m + e] *= cT;
-                S1[4 * m + e] *= cT;
+            for (int m = 0; m < IPT / 4; ++m) {
+                const ulonglong2 k = *(reinterpret_cast<const ulonglong2*>(s_k + j * DK + 32 * m) + part);
+                S0[2 * m] = f2_fma(k.x, ua[j], S0[2 * m]);
+                S1[2 * m] = f2_fma(k.x, ub[j], S1[2 * m]);
+                S0[2 * m + 1] = f2_fma(k.y, ua[j], S0[2 * m + 1]);
+                S1[2 * m + 1] = f2_fma(k.y, ub[j], S1[2 * m + 1]);
             }
-#pragma unroll
-            for (int j = 0; j < T; ++j) {
-                const float4 k = *(reinterpret_cast<const float4*>(s_k + j * DK + 32 * m) + part);
-                S0[4 * m] += k.x * ua[j];
-                S0[4 * m + 1] += k.y * ua[j];
-                S0[4 * m + 2] += k.z * ua[j];
-                S0[4 * m + 3] += k.w * ua[j];
-                S1[4 * m] += k.x * ub[j];
-                S1[4 * m + 1] += k.y * ub[j];
-                S1[4 * m + 2] += k.z * ub[j];
-                S1[4 * m + 3] += k.w * ub[j];
-            }
-        }
-        __syncthreads();                             // the small matrices and this stage may be written again
     }
     if (live) {
 #pragma unroll
-        for (int ii = 0; ii < IPT; ++ii) {
-            Sg[(size_t)(2 * ii) * stride + gt] = S0[ii];
-            Sg[(size_t)(2 * ii + 1) * stride + gt] = S1[ii];
+        for (int m = 0; m < IPT / 2; ++m) {
+            float* at = Sg + (size_t)(4 * m) * stride + gt;
+            f2_split(S0[m], at[0], at[2 * stride]);
+            f2_split(S1[m], at[stride], at[3 * stride]);
         }
     }
     // the kept inputs move on: this tile's value channels, and with the first tile the head's q and k channels
     // (every read of the old ones, here and in the prep kernel, is done)
     for (int e = tid; e < NC; e += DELTA_NT)
         if (col0 + e < p.dv)
-            move_kept(x0 + p.v_off + (size_t)h * p.dv + col0 + e, p.ld, kept + (size_t)(2 * p.dk + col0 + e) * (p.taps - 1), p.taps,
-                      len);
+            move_kept(v_src + e, p.ld, kept + (size_t)(2 * p.dk + col0 + e) * (p.taps - 1), p.taps, len);
     if (tile == 0)
         for (int e = tid; e < 2 * p.dk; e += DELTA_NT) {
             int col, wrow;
@@ -548,7 +630,7 @@ delta_chunk_kernel(const DeltaArgs p, const float* qn, const float* kn, const fl
 // ------------------------------------------------------------------ portions: unit norm per head, weight, gate
 template <typename TA>
 __global__ void __launch_bounds__(256)
-delta_out_kernel(const DeltaArgs p, const float* o, TA* out, int n) {
+delta_out_kernel(const DeltaArgs p, const float* o, TA* out, int n, int vec) {
     pdl_launch_dependents();
     pdl_wait();
     const size_t unit = (size_t)blockIdx.x * 8 + (threadIdx.x >> 5);
@@ -558,6 +640,31 @@ delta_out_kernel(const DeltaArgs p, const float* o, TA* out, int n) {
     const int h = (int)(unit - t * p.H);
     const float* row = o + unit * p.dv;
     const float* gate = p.rows + t * p.ld + p.g_off + (size_t)h * p.dv;
+    if (vec) {                                       // one group of four columns a lane
+        const int c = 4 * lane;
+        const bool in = c < p.dv;
+        const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+        float4 v = in ? *reinterpret_cast<const float4*>(row + c) : zero;
+        const float4 g = in && p.gate ? *reinterpret_cast<const float4*>(gate + c) : zero;
+        const float rs = 1.0f / sqrtf(warp_sum(v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w) / (float)p.dv + p.eps);
+        if (!in) return;
+        const float4 w = *reinterpret_cast<const float4*>(p.norm_w + c);
+        v.x *= rs * w.x * delta_gate_act(g.x, p.gate);
+        v.y *= rs * w.y * delta_gate_act(g.y, p.gate);
+        v.z *= rs * w.z * delta_gate_act(g.z, p.gate);
+        v.w *= rs * w.w * delta_gate_act(g.w, p.gate);
+        TA* dst = out + unit * p.dv + c;
+        if constexpr (sizeof(TA) == 4) {
+            *reinterpret_cast<float4*>(dst) = v;
+        } else {
+            __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+            uint2 q;
+            q.x = *reinterpret_cast<uint32_t*>(&a);
+            q.y = *reinterpret_cast<uint32_t*>(&b);
+            *reinterpret_cast<uint2*>(dst) = q;
+        }
+        return;
+    }
     float ss = 0.f;
     for (int c = lane; c < p.dv; c += 32) ss += row[c] * row[c];
     const float rs = 1.0f / sqrtf(warp_sum(ss) / (float)p.dv + p.eps);
@@ -592,33 +699,32 @@ static int launch_delta_step(const DeltaArgs& p, TA* out, cudaStream_t stream) {
     if (smem > 200 * 1024) return (int)cudaErrorInvalidValue;
     const int st = raise_smem(delta_step_kernel<TA, DK>, smem, raised);
     if (st) return st;
-    const int threads = p.dvp * 4 > 512 ? 512 : p.dvp * 4;              // a multiple of 32: dvp is a multiple of 8
+    const int most = delta_step_threads(DK), threads = p.dvp * 4 > most ? most : p.dvp * 4;      // a multiple of 32
     return rllm_launch(delta_step_kernel<TA, DK>, dim3(p.H, p.n_requests), dim3(threads), smem, stream, p, out);
 }
 
 template <int DK>
-static int launch_delta_chunk(const DeltaArgs& p, const float* qn, const float* kn, const float* prods, const float* bg,
-                              float* o, cudaStream_t stream) {
+static int launch_delta_chunk(const DeltaArgs& p, const float* qn, const float* kn, const float* mats, float* o,
+                              cudaStream_t stream) {
     static size_t raised = 0;
-    const int W = DELTA_TOK + p.taps - 1;
-    const size_t stage = 2 * DELTA_TOK * DK + DELTA_TOK * 16 + 2 * DELTA_TOK + (size_t)(W * DELTA_COLS + 3) / 4 * 4;
-    const size_t smem = (2 * stage + 2 * DELTA_TOK * DELTA_TOK + 2 * DELTA_TOK) * sizeof(float);
+    const size_t stage = 2 * DELTA_TOK * DK + DELTA_MAT + (size_t)(DELTA_TOK + p.taps - 1) * DELTA_COLS;
+    const size_t smem = 2 * stage * sizeof(float);
     if (smem > 200 * 1024) return (int)cudaErrorInvalidValue;
     const int st = raise_smem(delta_chunk_kernel<DK>, smem, raised);
     if (st) return st;
     const int n_tiles = (p.dvp + DELTA_COLS - 1) / DELTA_COLS;
-    return rllm_launch(delta_chunk_kernel<DK>, dim3(p.H * n_tiles, p.n_requests), dim3(DELTA_NT), smem, stream, p, qn, kn, prods,
-                       bg, o);
+    return rllm_launch(delta_chunk_kernel<DK>, dim3(p.H * n_tiles, p.n_requests), dim3(DELTA_NT), smem, stream, p, qn, kn, mats,
+                       o);
 }
 
-// portion 0: delta_step, the scratch arrays are not used; 1: prep, chunk, out (qn, kn [n, G * dk], prods [n, G, 16],
-// bg [n, H, 2], o [n, H * dv]).
+// portion 0: delta_step, the scratch arrays are not used; 1: prep, chunk, out (qn, kn [n, G * dk], mats [n / 8 + n_requests,
+// H, DELTA_MAT], o [n, H * dv]; all 16-byte aligned).
 RLLM_API int rllm_gated_delta(const float* rows, long long ld, int q_off, int k_off, int v_off, int g_off, int b_off,
                               int a_off, const float* conv, const float* A, const float* dt_bias, const float* norm_w,
                               float q_scale, float unit_eps, float eps, float* state, long long slot_stride,
                               const int* cu_q, const int* slots, void* out, int act_dt, int n, int n_requests, int H, int G,
-                              int dk, int dv, int taps, int gate_kind, int portion, float* qn, float* kn, float* prods,
-                              float* bg, float* o, cudaStream_t stream) {
+                              int dk, int dv, int taps, int gate_kind, int portion, float* qn, float* kn, float* mats,
+                              float* o, cudaStream_t stream) {
     if (n <= 0 || n_requests <= 0) return 0;
     if (H <= 0 || G <= 0 || H % G || dk <= 0 || dk > 512 || dv <= 0 || taps < 1 || taps > 64 || ld < (long long)q_off + G * dk)
         return (int)cudaErrorInvalidValue;
@@ -643,20 +749,26 @@ RLLM_API int rllm_gated_delta(const float* rows, long long ld, int q_off, int k_
         BY_DK(STEP);
 #undef STEP
     }
-    if (!qn || !kn || !prods || !bg || !o) return (int)cudaErrorInvalidValue;
-    const size_t smem = (size_t)2 * DELTA_TOK * dk * sizeof(float);
-    int st = rllm_launch(delta_prep_kernel, dim3(n / DELTA_TOK + n_requests, G), dim3(256), smem, stream, p, qn, kn, prods, bg);
+    if (!qn || !kn || !mats || !o) return (int)cudaErrorInvalidValue;
+    static size_t raised = 0;
+    const size_t smem = (size_t)DELTA_TOK * (2 * dk + 2 * (H / G)) * sizeof(float);
+    if (smem > 200 * 1024) return (int)cudaErrorInvalidValue;
+    int st = raise_smem(delta_prep_kernel, smem, raised);
+    if (st) return st;
+    st = rllm_launch(delta_prep_kernel, dim3(n / DELTA_TOK + n_requests, G), dim3(256), smem, stream, p, qn, kn, mats);
     if (st) return st;
     const auto chunks = [&]() -> int {
-#define CHUNK(D) launch_delta_chunk<D>(p, qn, kn, prods, bg, o, stream)
+#define CHUNK(D) launch_delta_chunk<D>(p, qn, kn, mats, o, stream)
         BY_DK(CHUNK);
 #undef CHUNK
     };
     st = chunks();
     if (st) return st;
     const dim3 grid((unsigned)(((size_t)n * H + 7) / 8));
-    if (act_dt == RLLM_F32) return rllm_launch(delta_out_kernel<float>, grid, dim3(256), 0, stream, p, (const float*)o, (float*)out, n);
-    return rllm_launch(delta_out_kernel<bf16>, grid, dim3(256), 0, stream, p, (const float*)o, (bf16*)out, n);
+    const int vec = dv <= 128 && (dv & 3) == 0 && (ld & 3) == 0 && (g_off & 3) == 0 && ((uintptr_t)rows & 15) == 0 &&
+                    ((uintptr_t)out & 15) == 0 && ((uintptr_t)norm_w & 15) == 0 && ((uintptr_t)o & 15) == 0;
+    if (act_dt == RLLM_F32) return rllm_launch(delta_out_kernel<float>, grid, dim3(256), 0, stream, p, (const float*)o, (float*)out, n, vec);
+    return rllm_launch(delta_out_kernel<bf16>, grid, dim3(256), 0, stream, p, (const float*)o, (bf16*)out, n, vec);
 }
 #undef BY_DK
 

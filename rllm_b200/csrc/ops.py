@@ -1008,14 +1008,14 @@ def gated_delta(rows, offs, conv, A, dt_bias, norm_w, q_scale, unit_eps, eps, st
     assert delta_state_floats(H, dk, dv, taps) <= st.shape[1]
     portion = max_q_len > DELTA_STEP_TOKENS
     new = lambda *s: torch.empty(s, dtype=torch.float32, device=out.device)
-    qn = kn = prods = bg = o = None
+    qn = kn = mats = o = None
     if portion:
-        qn, kn, prods, bg, o = new(n, G * dk), new(n, G * dk), new(n, G, 16), new(n, H, 2), new(n, H * dv)
+        qn, kn, mats, o = new(n, G * dk), new(n, G * dk), new(n // 8 + n_requests, H, 216), new(n, H * dv)
     _check(_lib("delta").rllm_gated_delta(
         _ptr(rows), c_longlong(rows.stride(0)), *(c_int(x) for x in offs), _ptr(conv), _ptr(A), _ptr(dt_bias), _ptr(norm_w),
         c_float(q_scale), c_float(unit_eps), c_float(eps), _ptr(st), c_longlong(st.stride(0)), _ptr(cu_q), _ptr(slots),
         _ptr(out), c_int(_code(out)), c_int(n), c_int(n_requests), c_int(H), c_int(G), c_int(dk), c_int(dv), c_int(taps),
-        c_int(GATES[gate]), c_int(1 if portion else 0), _ptr(qn), _ptr(kn), _ptr(prods), _ptr(bg), _ptr(o), _stream()),
+        c_int(GATES[gate]), c_int(1 if portion else 0), _ptr(qn), _ptr(kn), _ptr(mats), _ptr(o), _stream()),
         "gated_delta")
     if portion:
         global _launches
