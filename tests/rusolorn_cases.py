@@ -211,7 +211,7 @@ def marked_attention(cfg, w, asker, target, boost=6.0):
     return w
 
 
-def marked_delta(cfg, w, marker, gate=24.0, boost=4.0):
+def marked_delta(cfg, w, marker, gate=24.0, boost=30.0):
     """Layer 0: only the token `marker` writes (its write strength is nearly 1, the others' nearly 0) and nothing
     decays, so what the marker wrote is what the memory holds hundreds of tokens later: a state that is lost, reset
     or carried wrongly between steps and chunks changes every later row.  The stream's norm gets one column that is 1
