@@ -96,7 +96,10 @@ def weight_bytes(model):
     seen, total = set(), 0
     parts = [p for b in model.blocks for p in b.parts()] + [model.final_norm, model.lm_head]
     for p in parts:
+        parts += [v for v in vars(p).values() if hasattr(v, "expected_tensors")]        # parts made of parts
         for v in vars(p).values():
+            if getattr(v, "_base", None) is not None:
+                continue                                  # a view of a stacked matrix that is counted itself
             if hasattr(v, "data_ptr") and hasattr(v, "numel") and v.is_cuda and v.data_ptr() not in seen:
                 seen.add(v.data_ptr())
                 total += v.numel() * v.element_size()
@@ -244,12 +247,11 @@ def falalix_compare(a):
         width = widths[size]
         row = {}
         for name in (family, other):
-            fal = FAMILY_SHAPES[family](width)
+            fal = FAMILY_SHAPES[name if name in FAMILY_SHAPES else family](width)
             runs = len(fal["layers"])
             if fal.get("loop"):
                 runs += (fal["loop"]["stop"] - fal["loop"]["start"]) * (fal["loop"]["times"] - 1)
-            config = config_from_dict(fal if name == family else
-                                      FAMILY_SHAPES[other](width) if other in FAMILY_SHAPES else qwen3_shape(width, runs))
+            config = config_from_dict(fal if name in FAMILY_SHAPES else qwen3_shape(width, runs))
             model = random_model(config, seed=0, dtype="bfloat16", device="cuda:0", generate_on_device=True)
             V = model.spec.vocab_size
             eng = Engine(model, block_size=32, max_tokens=a.batch * (PROMPT + 256), max_requests=a.batch)

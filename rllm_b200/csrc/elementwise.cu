@@ -14,7 +14,7 @@
 // launch, this is the backstop.
 template <typename TW>
 __global__ void embed_kernel(const TW* __restrict__ table, const int* __restrict__ tokens,
-                             float* __restrict__ out, int d, int vocab, int* err) {
+                             float* __restrict__ out, int d, int vocab, float scale, int vec, int* err) {
     pdl_wait();
     pdl_launch_dependents();
     const int t = blockIdx.x;
@@ -25,16 +25,26 @@ __global__ void embed_kernel(const TW* __restrict__ table, const int* __restrict
     }
     const TW* src = table + (size_t)tok * d;
     float* dst = out + (size_t)t * d;
-    for (int i = threadIdx.x; i < d; i += blockDim.x) dst[i] = to_f<TW>(src[i]);
+    if (vec) {                                     // four columns a thread
+        for (int i = threadIdx.x * 4; i < d; i += blockDim.x * 4) {
+            struct alignas(4 * sizeof(TW)) Four { TW v[4]; };
+            const Four q = *reinterpret_cast<const Four*>(src + i);
+            *reinterpret_cast<float4*>(dst + i) = make_float4(to_f<TW>(q.v[0]) * scale, to_f<TW>(q.v[1]) * scale,
+                                                              to_f<TW>(q.v[2]) * scale, to_f<TW>(q.v[3]) * scale);
+        }
+        return;
+    }
+    for (int i = threadIdx.x; i < d; i += blockDim.x) dst[i] = to_f<TW>(src[i]) * scale;
 }
 
 RLLM_API int rllm_embed(const void* table, int table_dtype, const int* tokens, float* out, int n,
-                        int d, int vocab, int* err, cudaStream_t stream) {
+                        int d, int vocab, float scale, int* err, cudaStream_t stream) {
     if (n <= 0) return 0;
     const int threads = d >= 1024 ? 256 : 128;
+    const int vec = (d & 3) == 0 && ((uintptr_t)table & 15) == 0 && ((uintptr_t)out & 15) == 0;
     if (table_dtype == RLLM_F32)
-        return rllm_launch(embed_kernel<float>, dim3(n), dim3(threads), 0, stream, (const float*)table, tokens, out, d, vocab, err);
-    return rllm_launch(embed_kernel<bf16>, dim3(n), dim3(threads), 0, stream, (const bf16*)table, tokens, out, d, vocab, err);
+        return rllm_launch(embed_kernel<float>, dim3(n), dim3(threads), 0, stream, (const float*)table, tokens, out, d, vocab, scale, vec, err);
+    return rllm_launch(embed_kernel<bf16>, dim3(n), dim3(threads), 0, stream, (const bf16*)table, tokens, out, d, vocab, scale, vec, err);
 }
 
 // Embedding with a scale and a second table looked up by the pair (previous token, token):

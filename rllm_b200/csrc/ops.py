@@ -245,14 +245,14 @@ def core():
 
 # ------------------------------------------------------------------ elementwise
 
-def embed(table, tokens, out, err=None):
-    """out[t,:] = table[tokens[t],:] as float32.  table [V,d] f32/bf16, tokens int32 [n], out f32 [n,d]."""
+def embed(table, tokens, out, err=None, scale=1.0):
+    """out[t,:] = table[tokens[t],:] * scale as float32.  table [V,d] f32/bf16, tokens int32 [n], out f32 [n,d]."""
     _need_cuda(table, tokens, out)
     _need_contig(table=table, tokens=tokens, out=out)
     n, d = out.shape
     assert tokens.dtype == torch.int32 and out.dtype == torch.float32 and table.shape[1] == d
     _check(core().rllm_embed(_ptr(table), _code(table), _ptr(tokens), _ptr(out), c_int(n), c_int(d),
-                             c_int(table.shape[0]), _ptr(err), _stream()), "embed")
+                             c_int(table.shape[0]), c_float(scale), _ptr(err), _stream()), "embed")
     return out
 
 

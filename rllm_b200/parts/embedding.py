@@ -75,9 +75,7 @@ class Embedding(Part):
                            out, self.scale, self.buckets, self.mul_prev, self.mul_cur, ops.error_word(tokens.device))
             ops.keep_last_tokens(tokens, ctx.cu_q, cache.slots, last, ctx.n_requests)
             return out
-        ops.embed(self.weight, tokens, out, ops.error_word(tokens.device))
-        if self.scale != 1.0:
-            ops.axpby(self.scale, out, 0.0, out, out)
+        ops.embed(self.weight, tokens, out, ops.error_word(tokens.device), scale=self.scale)
         if self.norm_weight is not None:
             ops.norm_rows(out, self.norm_weight, self.norm_eps, x=out)       # in place
         return out
