@@ -239,8 +239,9 @@ delta_step_kernel(const DeltaArgs p, TA* out) {
 }
 
 // ------------------------------------------------------------------ portions: what a chunk needs beside the memory
-// Chunks are numbered through the step's requests in order.  qn, kn [n, G * dk]: the unit vectors (q times
-// q_scale).  mats [chunks, H, DELTA_MAT]: -beta_i d_ij (k_i . k_j) at [8 i + j], every entry twice (a pair that
+// Chunks are numbered through the step's requests in order; a chunk's rows lie together, eight of them whatever
+// the chunk holds, so that the chunk kernel fetches runs of memory.  qk [chunks, G, 2, 8, DK]: the unit vectors of q (times
+// q_scale) and k, zeros behind dk.  vals [chunks, H, 8, dvp]: the values behind their convolution.  mats [chunks, H, DELTA_MAT]: -beta_i d_ij (k_i . k_j) at [8 i + j], every entry twice (a pair that
 // multiplies two columns at once); d_ij (q_i . k_j) at [128 + 8 i + j] (0 for j > i); beta_i, c_i, d_8i at [192 + i], [200 + i],
 // [208 + i].  Tokens behind the last one of a short chunk have k = q = 0, beta = 0 and g = 1.
 #define DELTA_MAT 216
@@ -259,12 +260,32 @@ __device__ __forceinline__ float reduce16(const float (&a)[16], int lane) {
     return e + __shfl_xor_sync(0xffffffffu, e, 1);
 }
 
+// A channel's eight tokens behind its convolution (zeros behind the request's end): put(token, value).
+template <typename F>
+__device__ __forceinline__ void conv_chunk(const float* x, long long ld, const float* kept, const float* __restrict__ w,
+                                           int taps, int c0, int len, F put) {
+    if (taps == 4) {
+        float v[DELTA_TOK + 3];
+#pragma unroll
+        for (int j = 0; j < DELTA_TOK + 3; ++j) {
+            const int s = c0 + j - 3;
+            v[j] = s >= len ? 0.f : s >= 0 ? x[(size_t)s * ld] : kept[3 + s];
+        }
+        const float w0 = w[0], w1 = w[1], w2 = w[2], w3 = w[3];
+#pragma unroll
+        for (int i = 0; i < DELTA_TOK; ++i)
+            put(i, c0 + i < len ? silu_f(w0 * v[i] + w1 * v[i + 1] + w2 * v[i + 2] + w3 * v[i + 3]) : 0.f);
+    } else {
+        for (int i = 0; i < DELTA_TOK; ++i) put(i, c0 + i < len ? conv_at(x, ld, kept, w, taps, c0 + i) : 0.f);
+    }
+}
+
 __global__ void __launch_bounds__(256)
-delta_prep_kernel(const DeltaArgs p, float* qn, float* kn, float* mats) {
+delta_prep_kernel(const DeltaArgs p, float* qk, float* vals, float* mats, int DK) {
     extern __shared__ __align__(16) float sm_prep[];
-    float* s_q = sm_prep;                            // [TOK][dk]
-    float* s_k = s_q + DELTA_TOK * p.dk;
-    float* s_bg = s_k + DELTA_TOK * p.dk;            // [rep][2][TOK]: beta, g
+    float* s_q = sm_prep;                            // [TOK][DK]
+    float* s_k = s_q + DELTA_TOK * DK;
+    float* s_bg = s_k + DELTA_TOK * DK;              // [rep][2][TOK]: beta, g
     __shared__ float s_pr[DELTA_TOK][2 * DELTA_TOK]; // k_i . k_j, q_i . k_j
     // (no early launch of what follows: the chunk kernel's few, long-lived blocks are to spread over idle SMs)
     pdl_wait();
@@ -292,42 +313,43 @@ delta_prep_kernel(const DeltaArgs p, float* qn, float* kn, float* mats) {
         s_bg[hh * 2 * DELTA_TOK + i] = beta;
         s_bg[hh * 2 * DELTA_TOK + DELTA_TOK + i] = g;
     }
-    for (int c = tid; c < 2 * p.dk; c += blockDim.x) {       // a thread takes a channel's tokens
-        const bool is_k = c >= p.dk;
-        const int cc = is_k ? c - p.dk : c;
-        const float* x = x0 + (is_k ? p.k_off : p.q_off) + kh * p.dk + cc;
-        const float* w = p.conv + (size_t)((is_k ? p.G * p.dk : 0) + kh * p.dk + cc) * p.taps;
-        const float* kp = kept + (size_t)c * (p.taps - 1);
+    for (int e = tid; e < 2 * DK; e += blockDim.x) {         // a thread takes a channel's tokens
+        const bool is_k = e >= DK;
+        const int cc = is_k ? e - DK : e;
         float* dst = (is_k ? s_k : s_q) + cc;
-        if (p.taps == 4) {
-            float v[DELTA_TOK + 3];
-#pragma unroll
-            for (int j = 0; j < DELTA_TOK + 3; ++j) {
-                const int s = c0 + j - 3;
-                v[j] = s >= len ? 0.f : s >= 0 ? x[(size_t)s * p.ld] : kp[3 + s];
-            }
-            const float w0 = w[0], w1 = w[1], w2 = w[2], w3 = w[3];
-#pragma unroll
-            for (int i = 0; i < DELTA_TOK; ++i)
-                dst[i * p.dk] = silu_f(w0 * v[i] + w1 * v[i + 1] + w2 * v[i + 2] + w3 * v[i + 3]);
+        if (cc < p.dk) {
+            conv_chunk(x0 + (is_k ? p.k_off : p.q_off) + kh * p.dk + cc, p.ld, kept + (size_t)(is_k * p.dk + cc) * (p.taps - 1),
+                       p.conv + (size_t)((is_k ? p.G * p.dk : 0) + kh * p.dk + cc) * p.taps, p.taps, c0, len,
+                       [&](int i, float v) { dst[i * DK] = v; });
         } else {
-            for (int i = 0; i < cnt; ++i) dst[i * p.dk] = conv_at(x, p.ld, kp, w, p.taps, c0 + i);
+            for (int i = 0; i < DELTA_TOK; ++i) dst[i * DK] = 0.f;
+        }
+    }
+    for (int e = tid; e < rep * p.dvp; e += blockDim.x) {
+        const int hh = e / p.dvp, c = e - hh * p.dvp, h = kh * rep + hh;
+        float* dst = vals + ((size_t)blockIdx.x * p.H + h) * DELTA_TOK * p.dvp + c;
+        if (c < p.dv) {
+            conv_chunk(x0 + p.v_off + (size_t)h * p.dv + c, p.ld, kept + (size_t)(hh * C + 2 * p.dk + c) * (p.taps - 1),
+                       p.conv + (size_t)(2 * p.G * p.dk + h * p.dv + c) * p.taps, p.taps, c0, len,
+                       [&](int i, float v) { dst[(size_t)i * p.dvp] = v; });
+        } else {
+            for (int i = 0; i < DELTA_TOK; ++i) dst[(size_t)i * p.dvp] = 0.f;
         }
     }
     __syncthreads();
-    if (warp < cnt) {                                // warp i: token i's lengths
+    {                                                // warp i: token i's lengths
         const int i = warp;
         float qq = 0.f, kk = 0.f;
-        for (int c = lane; c < p.dk; c += 32) {
-            qq += s_q[i * p.dk + c] * s_q[i * p.dk + c];
-            kk += s_k[i * p.dk + c] * s_k[i * p.dk + c];
+        for (int c = lane; c < DK; c += 32) {
+            qq += s_q[i * DK + c] * s_q[i * DK + c];
+            kk += s_k[i * DK + c] * s_k[i * DK + c];
         }
         const float rq = p.q_scale / sqrtf(warp_sum(qq) + p.unit_eps), rk = 1.0f / sqrtf(warp_sum(kk) + p.unit_eps);
-        const size_t row = ((size_t)(t0 + c0 + i) * p.G + kh) * p.dk;
-        for (int c = lane; c < p.dk; c += 32) {
-            const float a = s_q[i * p.dk + c] * rq, b = s_k[i * p.dk + c] * rk;
-            s_q[i * p.dk + c] = qn[row + c] = a;
-            s_k[i * p.dk + c] = kn[row + c] = b;
+        float* row = qk + (((size_t)blockIdx.x * p.G + kh) * 2 * DELTA_TOK + i) * DK;
+        for (int c = lane; c < DK; c += 32) {
+            const float a = s_q[i * DK + c] * rq, b = s_k[i * DK + c] * rk;
+            s_q[i * DK + c] = row[c] = a;
+            s_k[i * DK + c] = row[(size_t)DELTA_TOK * DK + c] = b;
         }
     }
     __syncthreads();
@@ -336,16 +358,15 @@ delta_prep_kernel(const DeltaArgs p, float* qn, float* kn, float* mats) {
         float pr[16];
 #pragma unroll
         for (int j = 0; j < 16; ++j) pr[j] = 0.f;
-        if (i < cnt)
-            for (int c = lane; c < p.dk; c += 32) {
-                const float a = s_q[i * p.dk + c], b = s_k[i * p.dk + c];
+        for (int c = lane; c < DK; c += 32) {
+            const float a = s_q[i * DK + c], b = s_k[i * DK + c];
 #pragma unroll
-                for (int j = 0; j < DELTA_TOK; ++j) {
-                    const float o = j <= i ? s_k[j * p.dk + c] : 0.f;
-                    pr[j] += b * o;
-                    pr[DELTA_TOK + j] += a * o;
-                }
+            for (int j = 0; j < DELTA_TOK; ++j) {
+                const float o = j <= i ? s_k[j * DK + c] : 0.f;
+                pr[j] += b * o;
+                pr[DELTA_TOK + j] += a * o;
             }
+        }
         const float v = reduce16(pr, lane);
         if (!(lane & 1)) s_pr[i][lane >> 1] = v;
     }
@@ -413,16 +434,13 @@ __device__ __forceinline__ float reduce8(const f2 (&v)[DELTA_TOK], int part) {
     return (h1 ? c[1] : c[0]) + __shfl_xor_sync(0xffffffffu, h1 ? c[0] : c[1], 1);
 }
 
-#define DELTA_NT 128
-#define DELTA_COLS (2 * DELTA_NT / DELTA_PARTS)      // value columns of a block
-
-template <int DK>
-__global__ void __launch_bounds__(DELTA_NT)
-delta_chunk_kernel(const DeltaArgs p, const float* qn, const float* kn, const float* mats, float* o) {
-    constexpr int IPT = DK / DELTA_PARTS, T = DELTA_TOK, NC = DELTA_COLS, ROW4 = DK / 4;
+// A block of NT threads takes NT / 4 value columns.
+template <int DK, int NT>
+__global__ void __launch_bounds__(NT)
+delta_chunk_kernel(const DeltaArgs p, const float* qk, const float* vals, const float* mats, float* o) {
+    constexpr int IPT = DK / DELTA_PARTS, T = DELTA_TOK, NC = 2 * NT / DELTA_PARTS;
+    constexpr int QK4 = 2 * T * DK / 4, MAT4 = DELTA_MAT / 4, V4 = T * NC / 4, stage = 4 * (QK4 + MAT4 + V4);
     extern __shared__ __align__(16) float sm_chunk[];
-    const int W = T + p.taps - 1;                    // rows of the values' window
-    const int stage = 2 * T * DK + DELTA_MAT + W * NC;
     const int tid = threadIdx.x, part = tid & 7, lane = tid & 31;
     const int n_tiles = (p.dvp + NC - 1) / NC, h = blockIdx.x / n_tiles, tile = blockIdx.x % n_tiles, r = blockIdx.y;
     const int kh = h / (p.H / p.G), C = 2 * p.dk + p.dv;
@@ -435,12 +453,10 @@ delta_chunk_kernel(const DeltaArgs p, const float* qn, const float* kn, const fl
     float* slot = p.state + (size_t)p.slots[r] * p.slot_stride;
     float* Sg = slot + (size_t)h * DK * p.dvp;
     float* kept = slot + p.conv_base + (size_t)h * C * (p.taps - 1);
-    const float* kept_v = kept + (size_t)2 * p.dk * (p.taps - 1);
     const float* x0 = p.rows + (size_t)t0 * p.ld;
     const int col0 = tile * NC, pair = col0 / 2 + tid / DELTA_PARTS, gt = pair * DELTA_PARTS + part, cl = 2 * (tid / DELTA_PARTS);
     const bool live = 2 * pair < p.dvp;
     const size_t stride = (size_t)p.dvp * 4;
-    const bool vec = (p.dk & 3) == 0;
     f2 S0[IPT / 2], S1[IPT / 2];                     // rows ii, ii + 1 of the pair's two columns
 #pragma unroll
     for (int m = 0; m < IPT / 2; ++m) {
@@ -448,64 +464,37 @@ delta_chunk_kernel(const DeltaArgs p, const float* qn, const float* kn, const fl
         S0[m] = live ? f2_make(at[0], at[2 * stride]) : 0ull;
         S1[m] = live ? f2_make(at[stride], at[3 * stride]) : 0ull;
     }
-    // both stages start as zeros: the columns behind dk and behind dv are never filled
-    for (int e = tid; e < 2 * stage; e += DELTA_NT) sm_chunk[e] = 0.f;
-    __syncthreads();
-    const float* v_src = x0 + p.v_off + (size_t)h * p.dv + col0;
-    const size_t tok_stride = (size_t)p.G * p.dk;
-    const float* mat_src = mats + ((size_t)chunk0 * p.H + h) * DELTA_MAT;
-    auto fetch = [&](int c0, float* st) {
-        const int cnt = min(T, len - c0);
-        float *q = st, *k = st + T * DK, *m = k + T * DK, *v = m + DELTA_MAT;
-        const size_t src = (size_t)(t0 + c0) * tok_stride + (size_t)kh * p.dk;
-        if (vec) {
+    // a chunk's q and k, small matrices and values of this tile's columns: runs of 16 bytes
+    const float* qk_src = qk + ((size_t)chunk0 * p.G + kh) * 2 * T * DK + 4 * tid;
+    const float* mat_src = mats + ((size_t)chunk0 * p.H + h) * DELTA_MAT + 4 * tid;
+    const float* v_src = vals + ((size_t)chunk0 * p.H + h) * T * p.dvp + col0;
+    auto fetch = [&](float* st) {
 #pragma unroll
-            for (int it = 0; it < (T * ROW4 + DELTA_NT - 1) / DELTA_NT; ++it) {
-                const int e = tid + it * DELTA_NT, i = e / ROW4, c = 4 * (e % ROW4);
-                if (i < cnt && c < p.dk) {
-                    delta_cp16(q + i * DK + c, qn + src + i * tok_stride + c);
-                    delta_cp16(k + i * DK + c, kn + src + i * tok_stride + c);
-                }
-            }
-        } else {
-            for (int e = tid; e < cnt * DK; e += DELTA_NT) {
-                const int i = e / DK, c = e % DK;
-                if (c >= p.dk) continue;
-                delta_cp4(q + e, qn + src + i * tok_stride + c);
-                delta_cp4(k + e, kn + src + i * tok_stride + c);
-            }
+        for (int e = 0; e < QK4; e += NT) delta_cp16(st + 4 * (e + tid), qk_src + 4 * e);
+#pragma unroll
+        for (int e = 0; e < MAT4; e += NT)
+            if (e + tid < MAT4) delta_cp16(st + 4 * (QK4 + e + tid), mat_src + 4 * e);
+#pragma unroll
+        for (int e = tid; e < V4; e += NT) {
+            const int i = e / (NC / 4), c = 4 * (e % (NC / 4));
+            if (col0 + c < p.dvp) delta_cp16(st + 4 * (QK4 + MAT4 + e), v_src + (size_t)i * p.dvp + c);
         }
-        if (tid < DELTA_MAT / 4) delta_cp16(m + 4 * tid, mat_src + (size_t)(c0 / T) * p.H * DELTA_MAT + 4 * tid);
-        const int c = tid % NC;
-        if (col0 + c < p.dv)
-            for (int i = tid / NC; i < cnt + p.taps - 1; i += DELTA_NT / NC) {
-                const int s = c0 + i - (p.taps - 1);
-                delta_cp4(v + i * NC + c, s >= 0 ? v_src + (size_t)s * p.ld + c
-                                                 : kept_v + (size_t)(col0 + c) * (p.taps - 1) + p.taps - 1 + s);
-            }
         asm volatile("cp.async.commit_group;\n" ::);
+        qk_src += (size_t)p.G * 2 * T * DK;
+        mat_src += (size_t)p.H * DELTA_MAT;
+        v_src += (size_t)p.H * T * p.dvp;
     };
-    const float* wv0 = p.conv + (size_t)(2 * p.G * p.dk + h * p.dv + min(col0 + cl, p.dv - 1)) * p.taps;
-    const float* wv1 = p.conv + (size_t)(2 * p.G * p.dk + h * p.dv + min(col0 + cl + 1, p.dv - 1)) * p.taps;
-    float w4a[4] = {0.f, 0.f, 0.f, 0.f}, w4b[4] = {0.f, 0.f, 0.f, 0.f};       // the usual four taps stay in registers
-    if (p.taps == 4)
-#pragma unroll
-        for (int j = 0; j < 4; ++j) { w4a[j] = wv0[j]; w4b[j] = wv1[j]; }
     float* dst = o + ((size_t)(t0 + part) * p.H + h) * p.dv + col0 + cl;
     const bool st_a = col0 + cl < p.dv, st_b = col0 + cl + 1 < p.dv;
-    fetch(0, sm_chunk);
+    fetch(sm_chunk);
     int buf = 0;
     for (int c0 = 0; c0 < len; c0 += T, buf ^= 1) {
         const int cnt = min(T, len - c0);
         float* st = sm_chunk + buf * stage;
         asm volatile("cp.async.wait_group 0;\n" ::);
         __syncthreads();                             // this chunk is there, and everybody is done with the other stage
-        if (c0 + T < len) fetch(c0 + T, sm_chunk + (buf ^ 1) * stage);
+        if (c0 + T < len) fetch(sm_chunk + (buf ^ 1) * stage);
         float *s_q = st, *s_k = st + T * DK, *s_m = s_k + T * DK, *s_v = s_m + DELTA_MAT;
-        if (cnt < T) {                               // the last, short chunk: rows that an earlier chunk left here are cleared
-            for (int e = tid; e < (T - cnt) * DK; e += DELTA_NT) s_q[cnt * DK + e] = s_k[cnt * DK + e] = 0.f;
-            __syncthreads();
-        }
         f2 ka[T], kb[T], qa[T], qb[T];
 #pragma unroll
         for (int i = 0; i < T; ++i) ka[i] = kb[i] = qa[i] = qb[i] = 0ull;
@@ -536,26 +525,10 @@ delta_chunk_kernel(const DeltaArgs p, const float* qn, const float* kn, const fl
                 }
             }
         }
-        float va = 0.f, vb = 0.f;                    // this lane's token's values
-        if (p.taps == 4) {
-#pragma unroll
-            for (int j = 0; j < 4; ++j) {
-                const float2 x = *reinterpret_cast<const float2*>(s_v + (part + j) * NC + cl);
-                va += w4a[j] * x.x;
-                vb += w4b[j] * x.y;
-            }
-        } else {
-            for (int j = 0; j < p.taps; ++j) {
-                const float2 x = *reinterpret_cast<const float2*>(s_v + (part + j) * NC + cl);
-                va += wv0[j] * x.x;
-                vb += wv1[j] * x.y;
-            }
-        }
-        va = silu_f(va);
-        vb = silu_f(vb);
+        const float2 v = *reinterpret_cast<const float2*>(s_v + part * NC + cl);      // this lane's token's values
         const float ksa = reduce8(ka, part), ksb = reduce8(kb, part), qsa = reduce8(qa, part), qsb = reduce8(qb, part);
         const float beta = s_m[192 + part], c = s_m[200 + part];
-        const float ra = beta * (va - c * ksa), rb = beta * (vb - c * ksb);
+        const float ra = beta * (v.x - c * ksa), rb = beta * (v.y - c * ksb);
         f2 u[T];                                     // the tokens' corrections of the two columns
 #pragma unroll
         for (int i = 0; i < T; ++i)
@@ -616,11 +589,11 @@ delta_chunk_kernel(const DeltaArgs p, const float* qn, const float* kn, const fl
     }
     // the kept inputs move on: this tile's value channels, and with the first tile the head's q and k channels
     // (every read of the old ones, here and in the prep kernel, is done)
-    for (int e = tid; e < NC; e += DELTA_NT)
+    for (int e = tid; e < NC; e += NT)
         if (col0 + e < p.dv)
-            move_kept(v_src + e, p.ld, kept + (size_t)(2 * p.dk + col0 + e) * (p.taps - 1), p.taps, len);
+            move_kept(x0 + p.v_off + (size_t)h * p.dv + col0 + e, p.ld, kept + (size_t)(2 * p.dk + col0 + e) * (p.taps - 1), p.taps, len);
     if (tile == 0)
-        for (int e = tid; e < 2 * p.dk; e += DELTA_NT) {
+        for (int e = tid; e < 2 * p.dk; e += NT) {
             int col, wrow;
             head_channel(p, h, e, col, wrow);
             move_kept(x0 + col, p.ld, kept + (size_t)e * (p.taps - 1), p.taps, len);
@@ -704,26 +677,24 @@ static int launch_delta_step(const DeltaArgs& p, TA* out, cudaStream_t stream) {
 }
 
 template <int DK>
-static int launch_delta_chunk(const DeltaArgs& p, const float* qn, const float* kn, const float* mats, float* o,
+static int launch_delta_chunk(const DeltaArgs& p, const float* qk, const float* vals, const float* mats, float* o,
                               cudaStream_t stream) {
+    constexpr int NT = 64, NC = 2 * NT / DELTA_PARTS;           // measured: 64 threads ahead of 32 and 128 at every size
     static size_t raised = 0;
-    const size_t stage = 2 * DELTA_TOK * DK + DELTA_MAT + (size_t)(DELTA_TOK + p.taps - 1) * DELTA_COLS;
-    const size_t smem = 2 * stage * sizeof(float);
-    if (smem > 200 * 1024) return (int)cudaErrorInvalidValue;
-    const int st = raise_smem(delta_chunk_kernel<DK>, smem, raised);
+    const size_t smem = 2 * (2 * DELTA_TOK * DK + DELTA_MAT + DELTA_TOK * NC) * sizeof(float);
+    const int st = raise_smem(delta_chunk_kernel<DK, NT>, smem, raised);
     if (st) return st;
-    const int n_tiles = (p.dvp + DELTA_COLS - 1) / DELTA_COLS;
-    return rllm_launch(delta_chunk_kernel<DK>, dim3(p.H * n_tiles, p.n_requests), dim3(DELTA_NT), smem, stream, p, qn, kn, mats,
-                       o);
+    const int n_tiles = (p.dvp + NC - 1) / NC;
+    return rllm_launch(delta_chunk_kernel<DK, NT>, dim3(p.H * n_tiles, p.n_requests), dim3(NT), smem, stream, p, qk, vals, mats, o);
 }
 
-// portion 0: delta_step, the scratch arrays are not used; 1: prep, chunk, out (qn, kn [n, G * dk], mats [n / 8 + n_requests,
-// H, DELTA_MAT], o [n, H * dv]; all 16-byte aligned).
+// portion 0: delta_step, the scratch arrays are not used; 1: prep, chunk, out, with n / 8 + n_requests chunks in qk, vals
+// and mats (see the prep kernel) and o [n, H * dv]; all 16-byte aligned.
 RLLM_API int rllm_gated_delta(const float* rows, long long ld, int q_off, int k_off, int v_off, int g_off, int b_off,
                               int a_off, const float* conv, const float* A, const float* dt_bias, const float* norm_w,
                               float q_scale, float unit_eps, float eps, float* state, long long slot_stride,
                               const int* cu_q, const int* slots, void* out, int act_dt, int n, int n_requests, int H, int G,
-                              int dk, int dv, int taps, int gate_kind, int portion, float* qn, float* kn, float* mats,
+                              int dk, int dv, int taps, int gate_kind, int portion, float* qk, float* vals, float* mats,
                               float* o, cudaStream_t stream) {
     if (n <= 0 || n_requests <= 0) return 0;
     if (H <= 0 || G <= 0 || H % G || dk <= 0 || dk > 512 || dv <= 0 || taps < 1 || taps > 64 || ld < (long long)q_off + G * dk)
@@ -749,16 +720,16 @@ RLLM_API int rllm_gated_delta(const float* rows, long long ld, int q_off, int k_
         BY_DK(STEP);
 #undef STEP
     }
-    if (!qn || !kn || !mats || !o) return (int)cudaErrorInvalidValue;
+    if (!qk || !vals || !mats || !o) return (int)cudaErrorInvalidValue;
     static size_t raised = 0;
-    const size_t smem = (size_t)DELTA_TOK * (2 * dk + 2 * (H / G)) * sizeof(float);
+    const size_t smem = (size_t)DELTA_TOK * (2 * DK + 2 * (H / G)) * sizeof(float);
     if (smem > 200 * 1024) return (int)cudaErrorInvalidValue;
     int st = raise_smem(delta_prep_kernel, smem, raised);
     if (st) return st;
-    st = rllm_launch(delta_prep_kernel, dim3(n / DELTA_TOK + n_requests, G), dim3(256), smem, stream, p, qn, kn, mats);
+    st = rllm_launch(delta_prep_kernel, dim3(n / DELTA_TOK + n_requests, G), dim3(256), smem, stream, p, qk, vals, mats, DK);
     if (st) return st;
     const auto chunks = [&]() -> int {
-#define CHUNK(D) launch_delta_chunk<D>(p, qn, kn, mats, o, stream)
+#define CHUNK(D) launch_delta_chunk<D>(p, qk, vals, mats, o, stream)
         BY_DK(CHUNK);
 #undef CHUNK
     };

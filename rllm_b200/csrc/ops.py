@@ -979,11 +979,15 @@ def mlstm(rows, q_off, k_off, v_off, g_off, i_off, f_off, i_bias, f_bias, cap, q
 DELTA_STEP_TOKENS = 8         # steps in which no request brings more tokens than this take the token-by-token kernel
 
 
+def _delta_dk(dk: int) -> int:
+    """The key size the gated-delta kernels pad `dk` to."""
+    return next(s for s in (32, 64, 128, 256, 512) if dk <= s)
+
+
 def delta_state_floats(H: int, dk: int, dv: int, taps: int) -> int:
     """Floats of a request's gated-delta state: per head the dk x dv memory padded to the kernels' tile and in
     their threads' order, then per head the kept inputs of its convolutions (delta.cu).  No device needed."""
-    DK = next(s for s in (32, 64, 128, 256, 512) if dk <= s)
-    return H * DK * (-(-dv // 8) * 8) + H * (2 * dk + dv) * (taps - 1)
+    return H * _delta_dk(dk) * (-(-dv // 8) * 8) + H * (2 * dk + dv) * (taps - 1)
 
 
 def gated_delta(rows, offs, conv, A, dt_bias, norm_w, q_scale, unit_eps, eps, state, cu_q, slots, out, n_requests, max_q_len,
@@ -1008,14 +1012,16 @@ def gated_delta(rows, offs, conv, A, dt_bias, norm_w, q_scale, unit_eps, eps, st
     assert delta_state_floats(H, dk, dv, taps) <= st.shape[1]
     portion = max_q_len > DELTA_STEP_TOKENS
     new = lambda *s: torch.empty(s, dtype=torch.float32, device=out.device)
-    qn = kn = mats = o = None
+    qk = vals = mats = o = None
     if portion:
-        qn, kn, mats, o = new(n, G * dk), new(n, G * dk), new(n // 8 + n_requests, H, 216), new(n, H * dv)
+        chunks = n // 8 + n_requests
+        qk, vals = new(chunks, G, 2, 8, _delta_dk(dk)), new(chunks, H, 8, -(-dv // 8) * 8)
+        mats, o = new(chunks, H, 216), new(n, H * dv)
     _check(_lib("delta").rllm_gated_delta(
         _ptr(rows), c_longlong(rows.stride(0)), *(c_int(x) for x in offs), _ptr(conv), _ptr(A), _ptr(dt_bias), _ptr(norm_w),
         c_float(q_scale), c_float(unit_eps), c_float(eps), _ptr(st), c_longlong(st.stride(0)), _ptr(cu_q), _ptr(slots),
         _ptr(out), c_int(_code(out)), c_int(n), c_int(n_requests), c_int(H), c_int(G), c_int(dk), c_int(dv), c_int(taps),
-        c_int(GATES[gate]), c_int(1 if portion else 0), _ptr(qn), _ptr(kn), _ptr(mats), _ptr(o), _stream()),
+        c_int(GATES[gate]), c_int(1 if portion else 0), _ptr(qk), _ptr(vals), _ptr(mats), _ptr(o), _stream()),
         "gated_delta")
     if portion:
         global _launches
