@@ -122,6 +122,20 @@ static inline int rllm_launch(void (*kern)(KArgs...), dim3 grid, dim3 block, siz
     return (int)cudaLaunchKernelEx(&cfg, kern, static_cast<KArgs>(args)...);
 }
 
+// Without the attribute: the kernel starts when the one before has completed.  For kernels of many short
+// blocks that stream weights behind a kernel with few, long ones: launched early, their blocks would pile
+// up on whichever SMs have room at that moment and stay there while other SMs idle.
+template <typename... KArgs, typename... Args>
+static inline int rllm_launch_after(void (*kern)(KArgs...), dim3 grid, dim3 block, size_t smem, cudaStream_t stream,
+                                    Args... args) {
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = grid;
+    cfg.blockDim = block;
+    cfg.dynamicSmemBytes = smem;
+    cfg.stream = stream;
+    return (int)cudaLaunchKernelEx(&cfg, kern, static_cast<KArgs>(args)...);
+}
+
 // The same with the CTAs grouped into thread-block clusters of `cluster` CTAs along each dimension.
 template <typename... KArgs, typename... Args>
 static inline int rllm_launch_clusters(void (*kern)(KArgs...), dim3 grid, dim3 block, size_t smem, cudaStream_t stream,

@@ -500,7 +500,7 @@ RLLM_API int rllm_moe_expert_gate_up(const void* h, const void* w_gu, const int*
     if (d <= 0 || F <= 0 || top_k <= 0 || E <= 0 || !expert_kernels_fit(n, d) || ((uintptr_t)h & 15) || ((uintptr_t)w_gu & 15))
         return (int)cudaErrorInvalidValue;
     const GluForm glu = {limit, alpha, shift};
-    return rllm_launch(moe_expert_gate_up_kernel, dim3(E, (F + MOE_COLS - 1) / MOE_COLS), dim3(128), 0, stream,
+    return rllm_launch_after(moe_expert_gate_up_kernel, dim3(E, (F + MOE_COLS - 1) / MOE_COLS), dim3(128), 0, stream,
                        (const bf16*)h, (const bf16*)w_gu, idx, (bf16*)act, n * top_k, top_k, d, F, glu);
 }
 
@@ -510,7 +510,7 @@ RLLM_API int rllm_moe_expert_down(const void* act, const void* w_down, const int
     if (d <= 0 || F <= 0 || top_k <= 0 || E <= 0 || !expert_kernels_fit(n, F) || ((uintptr_t)act & 15) ||
         ((uintptr_t)w_down & 15))
         return (int)cudaErrorInvalidValue;
-    return rllm_launch(moe_expert_down_kernel, dim3(E, (d + MOE_DOWN_COLS - 1) / MOE_DOWN_COLS), dim3(128), 0, stream,
+    return rllm_launch_after(moe_expert_down_kernel, dim3(E, (d + MOE_DOWN_COLS - 1) / MOE_DOWN_COLS), dim3(128), 0, stream,
                        (const bf16*)act, (const bf16*)w_down, idx, y, n * top_k, d, F);
 }
 
