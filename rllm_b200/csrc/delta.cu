@@ -6,7 +6,7 @@
 // every channel over `taps` tokens (no bias, the last tap weighs the current token, zeros before the start):
 //   q = unit(silu(conv(q))) * q_scale,  k = unit(silu(conv(k))),  v = silu(conv(v)),  unit(x) = x / sqrt(sum x^2 + unit_eps)
 //   beta = sigmoid(b),  g = exp(-A * softplus(a + dt_bias))                        (A = exp(A_log), one per head)
-//   S <- g S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q
+//   w_t = beta_t (v_t - g_t M_(t-1)^T k_t),  M_t = g_t M_(t-1) + k_t w_t^T,  o_t = M_t^T q_t         (the code's S is M, its u is w)
 //   out = o / rms(o) * norm_w * act(gate)                                          (rms over the head's dv entries)
 // Everything here is float32; sums run in a fixed order, and who owns a state element is fixed by the sizes.
 //

@@ -9,10 +9,11 @@ head i uses query/key head floor(i / (H / G))):
         before the start) and silu
     q <- q / sqrt(sum q^2 + unit_eps) * q_scale,  k <- k / sqrt(sum k^2 + unit_eps)          per head
     beta = sigmoid(h Wb^T),  g = exp(-exp(A_log) softplus(h Wa^T + dt_bias))                 one each per value head
-    per head, S [dk, dv] zero before the first token:  S <- g S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q
+    per head, a memory M_t [dk, dv], M before the first token zero:
+        w_t = beta_t (v_t - g_t M_(t-1)^T k_t),   M_t = g_t M_(t-1) + k_t w_t^T,   o_t = M_t^T q_t
     out = ((o / rms(o) per head, eps inside the root, times norm [dv]) * gate(h Wg^T)) Wo^T
 
-State per request (float32): S of every head in the kernels' own order and the convolutions' last conv - 1
+State per request (float32): M of every head in the kernels' own order and the convolutions' last conv - 1
 inputs (csrc/delta.cu).  Parameters: hidden_size, num_heads, num_kv_heads, head_dim, v_head_dim, conv, q_scale, unit_eps,
 eps, gate ("silu", "sigmoid" or None).  Tensors under <prefix>: q, k [G*dk, d]; v, g [H*dv, d]; b, a [H, d]; q.conv, k.conv,
 v.conv [channels, conv]; A_log, dt_bias [H]; norm [dv]; o [d, H*dv].  q, k, v, the gate, b and a are one stacked product (rows

@@ -480,7 +480,7 @@ def test_token_by_token_and_portions(name, dtype):
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 @pytest.mark.parametrize("name", ["stack", "stack_other_order", "heads64", "heads128", "odd_sizes", "one_layer"])
 def test_unequal_requests_in_one_batch_with_reuse(name, dtype):
-    """Four requests of 70, 9, 31 and 2 tokens, portions of some beside single tokens of others, a fifth
+    """Four requests of 70, 9, 31 and 2 tokens, longer runs of one beside a decoded token of another, a fifth
     that takes over the pages and the slot of one that ended: every row is what the request gives alone."""
     cfg = CASES[name]
     w = rc.make_weights(cfg, 4, stored(dtype))
