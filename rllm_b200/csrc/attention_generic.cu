@@ -14,7 +14,8 @@
 // are the leading entries of the key rows themselves, v_cache == k_cache).
 // chunk > 0: positions are cut into runs of `chunk` counted from 0 and a token sees only the keys of
 // its own run (p >= pos - pos % chunk).  softcap > 0: a score s becomes softcap * tanh(s / softcap)
-// before the softmax.  sink (one number per query head, or null): the softmax's denominator also holds
+// before the softmax.  slopes (one number per query head, or null): slopes[h] * (pos - p) is taken off the score of
+// key p (behind the cap).  sink (one number per query head, or null): the softmax's denominator also holds
 // exp(sink[h]), which stands for no key and adds no value.
 //
 // Formula: crates/rllm-cpu/src/lib.rs:389-425 of AxiomOperator/rllm; its device
@@ -34,7 +35,8 @@ paged_attention_generic_kernel(const TQ* q, const TC* k_cache,
                                const int* __restrict__ positions, const int* __restrict__ seq_ids,
                                const int* __restrict__ block_table, int table_stride, int H, int K,
                                int hd, int hdv, int bs, float scale, int window, int keep_first, int n_pages,
-                               int* err, int chunk, float softcap, int v_ld, const float* __restrict__ sink) {
+                               int* err, int chunk, float softcap, int v_ld, const float* __restrict__ sink,
+                               const float* __restrict__ slopes) {
     extern __shared__ float smem[];
     pdl_wait();
     pdl_launch_dependents();
@@ -81,6 +83,7 @@ paged_attention_generic_kernel(const TQ* q, const TC* k_cache,
             for (int i = 0; i < hd; ++i) dot += qs[i] * to_f<TC>(kr[i]);
             s = dot * scale;
             if (softcap > 0.f) s = softcap * tanhf(s / softcap);
+            if (slopes) s -= slopes[h] * (float)(pos - p);
         }
         const float cmax = block_max(s, red);
         const float m_new = fmaxf(m_run, cmax);
@@ -118,7 +121,7 @@ RLLM_API int rllm_paged_attention_generic(const void* q, int q_dtype, const void
                                           const int* block_table, int table_stride, int n, int H,
                                           int K, int hd, int hdv, int bs, float scale, int window, int keep_first,
                                           int n_pages, int* err, int chunk, float softcap, int v_ld,
-                                          const float* sink, cudaStream_t stream) {
+                                          const float* sink, const float* slopes, cudaStream_t stream) {
     if (n <= 0) return 0;
     if (v_ld <= 0) v_ld = hdv;
     if (chunk < 0 || v_ld < hdv) return (int)cudaErrorInvalidValue;
@@ -132,11 +135,11 @@ RLLM_API int rllm_paged_attention_generic(const void* q, int q_dtype, const void
         return rllm_launch(paged_attention_generic_kernel<float, float, float>, grid, dim3(ATT_THREADS), smem,
                            stream, (const float*)q, (const float*)k_cache, (const float*)v_cache, (float*)out,
                            positions, seq_ids, block_table, table_stride, H, K, hd, hdv, bs, scale, window, keep_first, n_pages,
-                           err, chunk, softcap, v_ld, sink);
+                           err, chunk, softcap, v_ld, sink, slopes);
     return rllm_launch(paged_attention_generic_kernel<bf16, bf16, bf16>, grid, dim3(ATT_THREADS), smem, stream,
                        (const bf16*)q, (const bf16*)k_cache, (const bf16*)v_cache, (bf16*)out, positions,
                        seq_ids, block_table, table_stride, H, K, hd, hdv, bs, scale, window, keep_first, n_pages, err,
-                       chunk, softcap, v_ld, sink);
+                       chunk, softcap, v_ld, sink, slopes);
 }
 
 // the packed-argument forms (common.cuh) for the host runtime's replay of recorded launches

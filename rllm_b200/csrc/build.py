@@ -34,6 +34,7 @@ LIBRARIES = {
     "core": (["elementwise.cu", "rowwise.cu", "headwise.cu", "joins.cu", "attention_generic.cu", "gemm_plain.cu", "sampling.cu"], []),
     "recur": (["recurrent.cu"], []),
     "delta": (["delta.cu"], []),
+    "ssd": (["ssd.cu"], []),
     "moe": (["moe.cu"], []),
     "blas": (["gemm_lib.cu"], ["-lcublas"]),
     "fast": (["skinny_gemm.cu"], []),

@@ -10,7 +10,7 @@
 //                      square; queries out, keys into the paged cache; the values written beside them
 //                      are the key heads as projected (before rotation and norm), or the columns that
 //                      follow the keys when the row has them.
-//   latent_rope_store  one cache row per token [normed latent (rank) | rotated shared key part (r)],
+//   latent_rope_store  one cache row per token [normed latent (rank) | rotated shared key part (r, or none)],
 //                      and the rotated part of every query head copied behind that head's latent-space
 //                      query.
 //   head_norm_rope_store  per head of a [q | k | v] projection row: RMS norm with a weight, then the
@@ -271,7 +271,7 @@ RLLM_API int rllm_latent_rope_store(const void* q, int q_dt, long long ld_q, con
                                     int bs, float eps, int write_kv, long long n_slots, int* err, int pairs,
                                     cudaStream_t stream) {
     if (n <= 0) return 0;
-    if (H <= 0 || dq <= 0 || r <= 0 || (r & 1) || rank <= 0 || bs <= 0 || !cs_table || !kv_norm_w ||
+    if (H <= 0 || dq <= 0 || r < 0 || (r & 1) || rank <= 0 || bs <= 0 || (r && !cs_table) || !kv_norm_w ||
         ld_q < (long long)H * (dq + r) || ld_kv < rank + r)
         return (int)cudaErrorInvalidValue;
     const int ns = (int)(n_slots > 0x7fffffffLL ? 0x7fffffffLL : n_slots);

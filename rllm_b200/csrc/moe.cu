@@ -13,11 +13,14 @@
 //                    gate and up rows of four columns side by side (eight 16-byte loads in flight per lane).
 //   moe_pairs_down   out[t, c] = sum_j weight[t, j] * (Wd[e_j][c, :] . act[t * top_k + j, :]) in the order of j,
 //                    plus shared[t, c] * sigmoid(shared_gate[t]) when a shared expert's output is given.
+//   moe_pairs_up     the ungated form: act[pair, f] = f(weight[pair] * (Wu[e] . h[t])) with an activation by number; a weight
+//                    that multiplies an expert's input is a factor of its first product's result, so it is applied
+//                    there, in float32 (null: none).
 //   moe_sort         pairs counted per expert, offsets, and each pair's place in expert order (a stable
 //                    counting sort by one block); moe_gather_rows copies the tokens' rows into that order
 //                    and moe_combine adds a token's expert outputs back in the order of j.
 #include "common.cuh"
-#include <math.h>
+#include "activations.cuh"
 
 #define MOE_MAX_EXPERTS 1024
 #define MOE_MAX_TOP 32
@@ -237,6 +240,28 @@ moe_pairs_gate_up_kernel(const T* h, const T* __restrict__ w_gu, const int* idx,
     }
 }
 
+// h [n, d]; w_up [E][F][d]; act [n * top_k, F] = f(weight[pair] * (w_up[e] . h[t])); weight may be null
+template <typename T>
+__global__ void __launch_bounds__(256)
+moe_pairs_up_kernel(const T* h, const T* __restrict__ w_up, const int* idx, const float* weight, T* act, int top_k, int d, int F,
+                    int act_kind) {
+    extern __shared__ __align__(16) float s_h[];
+    pdl_wait();
+    pdl_launch_dependents();
+    const int pair = blockIdx.x, t = pair / top_k, e = idx[pair];
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    for (int i = threadIdx.x; i < d; i += blockDim.x) s_h[i] = to_f<T>(h[(size_t)t * d + i]);
+    __syncthreads();
+    const float wt = weight ? weight[pair] : 1.f;
+    const T* w = w_up + (size_t)e * F * d;
+    for (int c = warp; c < MOE_COLS; c += 8) {
+        const int f = blockIdx.y * MOE_COLS + c;
+        if (f >= F) break;
+        const float u = warp_sum(dot_row(w + (size_t)f * d, s_h, d, lane));
+        if (lane == 0) act[(size_t)pair * F + f] = from_f<T>(act_apply(wt * u, act_kind));
+    }
+}
+
 // act [n * top_k, F]; w_down [E][d][F]; out [n, d] float32; shared [n, d] float32 or null; gate: logits, one per token
 template <typename T>
 __global__ void __launch_bounds__(256)
@@ -266,7 +291,7 @@ moe_pairs_down_kernel(const T* act, const T* __restrict__ w_down, const int* idx
                     for (int jj = 0; jj < 4; ++jj) {
                         const int j = min(j0 + jj, top_k - 1);
                         const int e = idx[(size_t)t * top_k + j];
-                        wj[jj] = j0 + jj < top_k ? weight[(size_t)t * top_k + j] : 0.f;
+                        wj[jj] = j0 + jj < top_k ? (weight ? weight[(size_t)t * top_k + j] : 1.f) : 0.f;
                         rows[jj] = w_down + ((size_t)e * d + col0) * F;
                         rows[4 + jj] = w_down + ((size_t)e * d + c1) * F;
                         xs[jj] = s_a + (size_t)j * F;
@@ -307,7 +332,7 @@ moe_pairs_down_kernel(const T* act, const T* __restrict__ w_down, const int* idx
         for (int j = 0; j < top_k; ++j) {
             const int e = idx[(size_t)t * top_k + j];
             const float v = warp_sum(dot_row(w_down + ((size_t)e * d + col) * F, s_a + (size_t)j * F, F, lane));
-            sum += weight[(size_t)t * top_k + j] * v;
+            sum += (weight ? weight[(size_t)t * top_k + j] : 1.f) * v;
         }
         if (lane == 0) out[(size_t)t * d + col] = sum + (shared ? shared[(size_t)t * d + col] * sg : 0.f);
     }
@@ -324,6 +349,18 @@ RLLM_API int rllm_moe_pairs_gate_up(const void* h, const void* w_gu, int dt, con
                            (const float*)h, (const float*)w_gu, idx, (float*)act, top_k, d, F, glu);
     return rllm_launch(moe_pairs_gate_up_kernel<bf16>, grid, dim3(256), (size_t)d * sizeof(float), stream, (const bf16*)h,
                        (const bf16*)w_gu, idx, (bf16*)act, top_k, d, F, glu);
+}
+
+RLLM_API int rllm_moe_pairs_up(const void* h, const void* w_up, int dt, const int* idx, const float* weight, void* act, int n,
+                               int top_k, int d, int F, int act_kind, cudaStream_t stream) {
+    if (n <= 0) return 0;
+    if (d <= 0 || F <= 0 || top_k <= 0 || (size_t)d * sizeof(float) > 48 * 1024) return (int)cudaErrorInvalidValue;
+    const dim3 grid(n * top_k, (F + MOE_COLS - 1) / MOE_COLS);
+    if (dt == RLLM_F32)
+        return rllm_launch(moe_pairs_up_kernel<float>, grid, dim3(256), (size_t)d * sizeof(float), stream, (const float*)h,
+                           (const float*)w_up, idx, weight, (float*)act, top_k, d, F, act_kind);
+    return rllm_launch(moe_pairs_up_kernel<bf16>, grid, dim3(256), (size_t)d * sizeof(float), stream, (const bf16*)h,
+                       (const bf16*)w_up, idx, weight, (bf16*)act, top_k, d, F, act_kind);
 }
 
 RLLM_API int rllm_moe_pairs_down(const void* act, const void* w_down, int dt, const int* idx, const float* weight,
@@ -461,7 +498,37 @@ moe_expert_gate_up_kernel(const bf16* h, const bf16* __restrict__ w_gu, const in
     }
 }
 
-#define MOE_DOWN_COLS 64     // columns per block of the down product (4 warps, 16 columns a warp)
+#define MOE_DOWN_COLS 64     // columns per block of the products with one matrix (4 warps, 16 columns a warp)
+
+// act[pair, f] = f(weight[pair] * (Wu[e][f, :] . h[t])) for the pairs of the block's expert; a warp's 16 rows are 16 columns
+__global__ void __launch_bounds__(128)
+moe_expert_up_kernel(const bf16* h, const bf16* __restrict__ w_up, const int* idx, const float* weight, bf16* act, int n_pairs,
+                     int top_k, int d, int F, int act_kind) {
+    __shared__ int s_list[MOE_LIST];
+    __shared__ int s_n;
+    pdl_wait();
+    pdl_launch_dependents();
+    const int e = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, c = lane & 3;
+    const int cnt = list_expert_pairs(idx, n_pairs, e, s_list, &s_n);
+    if (cnt == 0) return;
+    const int f_lo = blockIdx.y * MOE_DOWN_COLS + warp * 16 + g, f_hi = f_lo + 8;
+    const bf16* lo = w_up + ((size_t)e * F + min(f_lo, F - 1)) * d;
+    const bf16* hi = w_up + ((size_t)e * F + min(f_hi, F - 1)) * d;
+    for (int c0 = 0; c0 < cnt; c0 += MOE_MT) {
+        const int mine = s_list[min(c0 + g, cnt - 1)];
+        float acc[4];
+        rows16_times_tokens8(lo, hi, h + (size_t)(mine / top_k) * d, d, c, acc);
+#pragma unroll
+        for (int q = 0; q < 2; ++q) {
+            const int at = c0 + 2 * c + q;
+            if (at >= cnt) continue;
+            const size_t pair = s_list[at];
+            const float wt = weight ? weight[pair] : 1.f;
+            if (f_lo < F) act[pair * F + f_lo] = from_f<bf16>(act_apply(wt * acc[q], act_kind));
+            if (f_hi < F) act[pair * F + f_hi] = from_f<bf16>(act_apply(wt * acc[2 + q], act_kind));
+        }
+    }
+}
 
 // y[pair, col] = Wd[e][col, :] . act[pair, :] for the pairs of the block's expert; moe_combine weights and adds them
 __global__ void __launch_bounds__(128)
@@ -502,6 +569,15 @@ RLLM_API int rllm_moe_expert_gate_up(const void* h, const void* w_gu, const int*
     const GluForm glu = {limit, alpha, shift};
     return rllm_launch_after(moe_expert_gate_up_kernel, dim3(E, (F + MOE_COLS - 1) / MOE_COLS), dim3(128), 0, stream,
                        (const bf16*)h, (const bf16*)w_gu, idx, (bf16*)act, n * top_k, top_k, d, F, glu);
+}
+
+RLLM_API int rllm_moe_expert_up(const void* h, const void* w_up, const int* idx, const float* weight, void* act, int n, int top_k,
+                                int E, int d, int F, int act_kind, cudaStream_t stream) {
+    if (n <= 0) return 0;
+    if (d <= 0 || F <= 0 || top_k <= 0 || E <= 0 || !expert_kernels_fit(n, d) || ((uintptr_t)h & 15) || ((uintptr_t)w_up & 15))
+        return (int)cudaErrorInvalidValue;
+    return rllm_launch_after(moe_expert_up_kernel, dim3(E, (F + MOE_DOWN_COLS - 1) / MOE_DOWN_COLS), dim3(128), 0, stream,
+                             (const bf16*)h, (const bf16*)w_up, idx, weight, (bf16*)act, n * top_k, top_k, d, F, act_kind);
 }
 
 RLLM_API int rllm_moe_expert_down(const void* act, const void* w_down, const int* idx, float* y, int n, int top_k, int E,
@@ -569,10 +645,15 @@ RLLM_API int rllm_moe_sort(const int* idx, int n_pairs, int E, int* offsets, int
 // rows allow it) and writes it to the places of its top_k pairs
 template <typename T>
 __global__ void __launch_bounds__(256)
-moe_gather_rows_kernel(const T* h, const int* __restrict__ place, T* rows, int top_k, int d, int vec) {
+moe_gather_rows_kernel(const T* h, const int* __restrict__ place, T* rows, int top_k, int d, int vec, const float* weight,
+                       float* weight_out) {
     pdl_wait();
     pdl_launch_dependents();
     const int t = blockIdx.x;
+    if (weight_out && (int)threadIdx.x < top_k) {
+        const size_t p = (size_t)t * top_k + threadIdx.x;
+        weight_out[place[p]] = weight[p];
+    }
     const T* src = h + (size_t)t * d;
     if (vec) {
         const int n16 = (int)((size_t)d * sizeof(T) / 16);
@@ -591,17 +672,17 @@ moe_gather_rows_kernel(const T* h, const int* __restrict__ place, T* rows, int t
 }
 
 RLLM_API int rllm_moe_gather_rows(const void* h, int dt, const int* place, void* rows, int n_pairs, int top_k, int d,
-                                  cudaStream_t stream) {
+                                  const float* weight, float* weight_out, cudaStream_t stream) {
     if (n_pairs <= 0) return 0;
-    if (top_k <= 0 || n_pairs % top_k) return (int)cudaErrorInvalidValue;
+    if (top_k <= 0 || n_pairs % top_k || (weight_out && (!weight || top_k > 128))) return (int)cudaErrorInvalidValue;
     const size_t row_bytes = (size_t)d * (dt == RLLM_F32 ? 4 : 2);
     const int vec = row_bytes % 16 == 0 && ((uintptr_t)h & 15) == 0 && ((uintptr_t)rows & 15) == 0;
     const dim3 grid(n_pairs / top_k), block(row_bytes >= 4096 ? 256 : 128);
     if (dt == RLLM_F32)
         return rllm_launch(moe_gather_rows_kernel<float>, grid, block, 0, stream, (const float*)h, place, (float*)rows,
-                           top_k, d, vec);
+                           top_k, d, vec, weight, weight_out);
     return rllm_launch(moe_gather_rows_kernel<bf16>, grid, block, 0, stream, (const bf16*)h, place, (bf16*)rows, top_k, d,
-                       vec);
+                       vec, weight, weight_out);
 }
 
 // out[t] = sum_j weight[t, j] * y[place[t * top_k + j]] (+ shared[t] * sigmoid(gate[t])); place null: y in pair order
@@ -622,7 +703,7 @@ moe_combine_kernel(const float* y, const int* place, const float* weight, float*
     for (int v = 0; v < VEC; ++v) sum[v] = 0.f;
 #pragma unroll 4
     for (int j = 0; j < top_k; ++j) {
-        const float w = weight[(size_t)t * top_k + j];
+        const float w = weight ? weight[(size_t)t * top_k + j] : 1.f;
         const float* row = y + (size_t)(place ? place[(size_t)t * top_k + j] : t * top_k + j) * d + i;
         if constexpr (VEC == 4) {
             const float4 r = *reinterpret_cast<const float4*>(row);
@@ -661,6 +742,8 @@ RLLM_API int rllm_moe_combine(const float* y, const int* place, const float* wei
 RLLM_PACKED(rllm_moe_route)
 RLLM_PACKED(rllm_moe_pairs_gate_up)
 RLLM_PACKED(rllm_moe_pairs_down)
+RLLM_PACKED(rllm_moe_pairs_up)
+RLLM_PACKED(rllm_moe_expert_up)
 RLLM_PACKED(rllm_moe_expert_gate_up)
 RLLM_PACKED(rllm_moe_expert_down)
 RLLM_PACKED(rllm_moe_sort)

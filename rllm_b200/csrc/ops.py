@@ -369,14 +369,16 @@ def qk_norm_rope_store(qkv, q_norm_w, k_norm_w, inv_freq, positions, slots, q_ou
 
 def paged_attention_generic(q, k_cache, v_cache, out, positions, seq_ids, block_table, H, K, hd,
                             block_size, scale, window=0, keep_first=0, v_head_dim=None, chunk=0, softcap=0.0,
-                            sink=None):
+                            sink=None, slopes=None):
     """Plain paged causal attention; q [n, H*hd], out [n, H*hdv], caches [pages, K, block_size, hd] and
     [pages, K, block_size, hdv] (hdv = v_head_dim, hd by default).  keep_first: the first keys of a
     request stay visible when the window has passed them.  chunk: a token sees only the keys of its
     own run of that many positions (counted from 0).  softcap: scores go through cap * tanh(s / cap).
     `v_cache is k_cache` with hdv < hd: the values are the first hdv entries of the key rows.
-    sink (float32 [H]): exp(sink[h]) joins the softmax's denominator of head h, with no key and no value."""
-    _need_cuda(q, k_cache, v_cache, out, positions, seq_ids, block_table, sink)
+    sink (float32 [H]): exp(sink[h]) joins the softmax's denominator of head h, with no key and no value.
+    slopes (float32 [H]): slopes[h] * (i - j) is taken off the score of the query at i and the key at j."""
+    _need_cuda(q, k_cache, v_cache, out, positions, seq_ids, block_table, sink, slopes)
+    assert slopes is None or (slopes.dtype == torch.float32 and slopes.numel() == H and slopes.is_contiguous())
     assert sink is None or (sink.dtype == torch.float32 and sink.numel() == H and sink.is_contiguous())
     _need_contig(q=q, k_cache=k_cache, v_cache=v_cache, out=out, positions=positions, seq_ids=seq_ids)
     n = q.shape[0]
@@ -395,7 +397,7 @@ def paged_attention_generic(q, k_cache, v_cache, out, positions, seq_ids, block_
         c_int(_code(out)), _ptr(positions), _ptr(seq_ids), _ptr(block_table), c_int(block_table.stride(0)),
         c_int(n), c_int(H), c_int(K), c_int(hd), c_int(hdv), c_int(block_size), c_float(scale), c_int(window),
         c_int(keep_first), c_int(min(k_cache.shape[0], 0x7fffffff)), _ptr(error_word(q.device)), c_int(chunk),
-        c_float(softcap), c_int(v_ld), _ptr(sink), _stream()),
+        c_float(softcap), c_int(v_ld), _ptr(sink), _ptr(slopes), _stream()),
         "paged_attention_generic")
     return out
 
@@ -581,7 +583,7 @@ def latent_rope_store(q, kv, kv_norm_w, cs_table, cs_mult, slots, q_att, cache, 
     """Attention through latents, the step between the projections and the attention kernel: kv
     [n, rank + r] (float32, any row stride) -> cache row [normed latent | rotated shared key part];
     q [n, H * (dq + r)] -> the rotated part of every head into q_att[:, h, rank:rank + r].  `pairs`: entry 2i
-    turns with 2i + 1 (else i with i + r/2).  See headwise.cu."""
+    turns with 2i + 1 (else i with i + r/2).  r 0: no rotated parts, no cs_table.  See headwise.cu."""
     _need_cuda(q, kv, kv_norm_w, cs_table, slots, q_att, cache)
     _need_contig(q_att=q_att, cache=cache, slots=slots)
     _rows2d(q, "q"), _rows2d(kv, "kv")
@@ -590,7 +592,7 @@ def latent_rope_store(q, kv, kv_norm_w, cs_table, cs_mult, slots, q_att, cache, 
     assert q_att.shape == (n, H * (rank + r)) and cache.shape[1:] == (1, block_size, rank + r)
     assert cache.dtype == q_att.dtype and slots.dtype == torch.int32 and slots.numel() == n
     assert kv_norm_w.dtype == torch.float32 and kv_norm_w.numel() == rank and kv_norm_w.is_contiguous()
-    assert cs_table.dtype == torch.float32 and cs_table.shape == (n, r // 2, 2) and cs_table.is_contiguous()
+    assert r == 0 or (cs_table.dtype == torch.float32 and cs_table.shape == (n, r // 2, 2) and cs_table.is_contiguous())
     _check(core().rllm_latent_rope_store(
         _ptr(q), c_int(_code(q)), c_longlong(q.stride(0)), _ptr(kv), c_longlong(kv.stride(0)), _ptr(kv_norm_w),
         _ptr(cs_table), c_float(cs_mult), _ptr(slots), _ptr(q_att), _ptr(cache), c_int(_code(q_att)), c_int(n),
@@ -638,8 +640,8 @@ def _rows2d(t, name):
     return t
 
 
-def rows_act(a, out, act=None, bias=None, mul=None, mul_act=None, mul_group=1):
-    """out[t, c] = f(a[t, c] + bias[c]) * g(mul[t, c // mul_group]); a, mul, out may be column slices of
+def rows_act(a, out, act=None, bias=None, mul=None, mul_act=None, mul_group=1, factor=1.0, row_scale=None):
+    """out[t, c] = factor * f(row_scale[t] * a[t, c] + bias[c]) * g(mul[t, c // mul_group]); row_scale float32 [n] or None; a, mul, out may be column slices of
     wider matrices (any row stride), float32 or bfloat16; bias float32.  f, g by name (ACT).  mul_group > 1:
     one factor for each run of that many columns (a gate per head)."""
     _need_cuda(a, out, bias, mul)
@@ -648,11 +650,12 @@ def rows_act(a, out, act=None, bias=None, mul=None, mul_act=None, mul_group=1):
     assert mul_group >= 1 and cols % mul_group == 0
     assert a.shape == (n, cols) and (mul is None or _rows2d(mul, "mul").shape == (n, cols // mul_group))
     assert bias is None or (bias.dtype == torch.float32 and bias.numel() == cols and bias.is_contiguous())
+    assert row_scale is None or (row_scale.dtype == torch.float32 and row_scale.numel() == n and row_scale.is_contiguous())
     _check(core().rllm_rows_act(_ptr(a), c_int(_code(a)), c_longlong(a.stride(0)), _ptr(bias), c_int(ACT[act]),
                                 _ptr(mul), c_int(_code(mul) if mul is not None else F32),
                                 c_longlong(mul.stride(0) if mul is not None else 0), c_int(ACT[mul_act]), _ptr(out),
                                 c_int(_code(out)), c_longlong(out.stride(0)), c_int(n), c_int(cols), c_int(mul_group),
-                                _stream()), "rows_act")
+                                c_float(factor), _ptr(row_scale), _stream()), "rows_act")
     return out
 
 
@@ -1029,6 +1032,53 @@ def gated_delta(rows, offs, conv, A, dt_bias, norm_w, q_scale, unit_eps, eps, st
     return out
 
 
+SSD_STEP_TOKENS = 8           # steps in which no request brings more tokens than this take one kernel (SSD_STEP in ssd.cu)
+
+
+def ssd_state_floats(H: int, P: int, N: int, G: int, taps: int) -> int:
+    """Floats of a request's state: S of every head [H][P][N], then the ring of the convolution's last inputs (ssd.cu), rounded
+    up to a multiple of 4 each.  No device needed."""
+    return (H * P * N + (taps - 1 + SSD_STEP_TOKENS) * (H * P + 2 * G * N) + 3) // 4 * 4
+
+
+def ssd(rows, conv, conv_b, dt_bias, A, D, norm_w, eps, norm_groups, state, ctx, slots, out, H, G, P, N):
+    """The state-space recurrence with one decay per head behind its convolution, gated and normed; see ssd.cu.  rows: float32
+    [n, ...] with z [H*P], the convolution's channels x [H*P], B, C [G*N] each, and dt [H] side by side; conv float32 [taps,
+    channels]; dt_bias, A (exp of the stored logarithms), D float32 [H]; norm_w float32 [H*P]; ctx: the step's StepContext; out
+    activation type [n, H*P], any row stride."""
+    _need_cuda(rows, conv, conv_b, dt_bias, A, D, norm_w, state, slots, out)
+    _rows2d(rows, "rows"), _rows2d(out, "out")
+    _need_contig(conv=conv, conv_b=conv_b, dt_bias=dt_bias, A=A, D=D, norm_w=norm_w)
+    n, taps, inner, C = out.shape[0], conv.shape[0], H * P, H * P + 2 * G * N
+    assert rows.dtype == torch.float32 and rows.shape[0] == n and rows.shape[1] >= inner + C + H and out.shape == (n, inner)
+    assert conv.shape == (taps, C) and conv_b.numel() == C and dt_bias.numel() == A.numel() == D.numel() == H
+    assert norm_w.numel() == inner and inner % norm_groups == 0
+    for w in (conv, conv_b, dt_bias, A, D, norm_w):
+        assert w.dtype == torch.float32
+    if N > 256:
+        raise KernelError(f"ssd: at most 256 state entries per column, got {N}")
+    st = _state2d(state)
+    assert ssd_state_floats(H, P, N, G, taps) <= st.shape[1]
+    mode, xbc, dts, ldx = 0, None, None, 0
+    if ctx.max_q_len > SSD_STEP_TOKENS:
+        mode = 2 if out.dtype == torch.bfloat16 else 1
+        ldx = H * (-(-P // 8) * 8) + 2 * G * (-(-N // 8) * 8)
+        make = torch.empty if P % 8 == 0 and N % 8 == 0 else torch.zeros       # padding entries of a head or group read as zero
+        xbc = make((n, ldx), dtype=out.dtype, device=out.device)
+        dts = torch.empty((2, H, n), dtype=torch.float32, device=out.device)
+    _check(_lib("ssd").rllm_ssd(
+        _ptr(rows), c_longlong(rows.stride(0)), c_int(0), c_int(inner), c_int(inner + C), _ptr(conv), _ptr(conv_b), _ptr(dt_bias),
+        _ptr(A), _ptr(D), _ptr(st), c_longlong(st.stride(0)), _ptr(ctx.positions), _ptr(ctx.seq_ids), _ptr(ctx.cu_q), _ptr(slots),
+        c_int(H), c_int(G), c_int(P), c_int(N), c_int(taps), c_int(n), c_int(ctx.n_requests), c_int(mode), _ptr(xbc),
+        c_longlong(ldx), _ptr(dts), _ptr(out), c_int(_code(out)), c_longlong(out.stride(0)), _stream()), "ssd")
+    _check(_lib("ssd").rllm_ssd_norm(_ptr(out), c_int(_code(out)), c_longlong(out.stride(0)), _ptr(norm_w), c_int(n),
+                                     c_int(norm_groups), c_int(inner // norm_groups), c_float(eps), _stream()), "ssd_norm")
+    if mode:
+        global _launches
+        _launches += 1                         # the convolution's kernel
+    return out
+
+
 # ------------------------------------------------------------------ routed experts (moe.cu)
 
 def moe_route(logits, correction, idx, weight, E, top_k, n_groups=1, keep_groups=1, group_best=2, score="sigmoid",
@@ -1084,8 +1134,27 @@ def moe_pairs_gate_up(h, w_gu, idx, act, glu=(0.0, 1.0, 0.0)):
     return act
 
 
+def moe_pairs_up(h, w_up, idx, weight, act, activation):
+    """act[t * top_k + j] = f(weight[t, j] * (Wu[e] h[t])) with e = idx[t, j] (weight None: no factor); w_up [E, F, d]; h, w_up,
+    act of one type; f by name (ACT).  Which way it runs: as moe_pairs_gate_up."""
+    _need_cuda(h, w_up, idx, weight, act)
+    _need_contig(h=h, w_up=w_up, idx=idx, weight=weight, act=act)
+    n, d = h.shape
+    top_k, F = idx.shape[1], act.shape[1]
+    assert w_up.shape[1:] == (F, d) and act.shape == (n * top_k, F) and h.dtype == w_up.dtype == act.dtype
+    assert weight is None or (weight.dtype == torch.float32 and weight.shape == (n, top_k))
+    if _by_expert(h, n, d):
+        _check(_lib("moe").rllm_moe_expert_up(_ptr(h), _ptr(w_up), _ptr(idx), _ptr(weight), _ptr(act), c_int(n), c_int(top_k),
+                                              c_int(w_up.shape[0]), c_int(d), c_int(F), c_int(ACT[activation]), _stream()),
+               "moe_expert_up")
+        return act
+    _check(_lib("moe").rllm_moe_pairs_up(_ptr(h), _ptr(w_up), c_int(_code(h)), _ptr(idx), _ptr(weight), _ptr(act), c_int(n),
+                                         c_int(top_k), c_int(d), c_int(F), c_int(ACT[activation]), _stream()), "moe_pairs_up")
+    return act
+
+
 def moe_pairs_down(act, w_down, idx, weight, out, shared=None, gate=None):
-    """out[t] = sum_j weight[t, j] * Wd[idx[t, j]] act[t * top_k + j] (+ shared[t] * sigmoid(gate[t]));
+    """out[t] = sum_j weight[t, j] (weight None: 1) * Wd[idx[t, j]] act[t * top_k + j] (+ shared[t] * sigmoid(gate[t]));
     w_down [E, d, F]; out, shared float32 [n, d]; gate: float32 logits, one per token (a column)."""
     _need_cuda(act, w_down, idx, weight, out, shared, gate)
     _need_contig(act=act, w_down=w_down, idx=idx, weight=weight, out=out, shared=shared)
@@ -1098,7 +1167,7 @@ def moe_pairs_down(act, w_down, idx, weight, out, shared=None, gate=None):
         y = torch.empty((n * top_k, d), dtype=torch.float32, device=out.device)
         _check(_lib("moe").rllm_moe_expert_down(_ptr(act), _ptr(w_down), _ptr(idx), _ptr(y), c_int(n), c_int(top_k),
                                                 c_int(w_down.shape[0]), c_int(d), c_int(F), _stream()), "moe_expert_down")
-        return moe_combine(y, None, weight, out, shared, gate)
+        return moe_combine(y, None, weight, out, shared, gate, top_k)
     if top_k * F * 4 > 96 * 1024:
         raise KernelError("moe_pairs_down: top_k * expert size exceeds the kernel's shared memory")
     _check(_lib("moe").rllm_moe_pairs_down(_ptr(act), _ptr(w_down), c_int(_code(act)), _ptr(idx), _ptr(weight), _ptr(out),
@@ -1118,23 +1187,26 @@ def moe_sort(idx, E):
     return offsets, place
 
 
-def moe_gather_rows(h, place, rows, top_k):
-    """rows[place[p]] = h[p // top_k] for every pair p."""
-    _need_cuda(h, place, rows)
-    _need_contig(h=h, place=place, rows=rows)
+def moe_gather_rows(h, place, rows, top_k, weight=None, weight_out=None):
+    """rows[place[p]] = h[p // top_k] for every pair p, and weight_out[place[p]] = weight[p] if given."""
+    _need_cuda(h, place, rows, weight, weight_out)
+    _need_contig(h=h, place=place, rows=rows, weight=weight, weight_out=weight_out)
+    assert weight_out is None or (weight.dtype == weight_out.dtype == torch.float32 and weight.numel() == weight_out.numel()
+                                  == place.numel())
     assert rows.shape == (place.numel(), h.shape[1]) and rows.dtype == h.dtype
     _check(_lib("moe").rllm_moe_gather_rows(_ptr(h), c_int(_code(h)), _ptr(place), _ptr(rows), c_int(place.numel()),
-                                            c_int(top_k), c_int(h.shape[1]), _stream()), "moe_gather_rows")
+                                            c_int(top_k), c_int(h.shape[1]), _ptr(weight), _ptr(weight_out), _stream()),
+           "moe_gather_rows")
     return rows
 
 
-def moe_combine(y, place, weight, out, shared=None, gate=None):
+def moe_combine(y, place, weight, out, shared=None, gate=None, top_k=None):
     """out[t] = sum_j weight[t, j] * y[place[t * top_k + j]] (+ shared[t] * sigmoid(gate[t])), float32;
-    place None: y holds the pairs in their own order."""
+    place None: y holds the pairs in their own order.  weight None: every weight is 1 (`top_k` is then needed)."""
     _need_cuda(y, place, weight, out, shared, gate)
     _need_contig(y=y, place=place, weight=weight, out=out, shared=shared)
     n, d = out.shape
-    top_k = weight.shape[1]
+    top_k = weight.shape[1] if weight is not None else int(top_k)
     assert y.dtype == out.dtype == torch.float32 and y.shape == (n * top_k, d)
     assert shared is None or (shared.dtype == torch.float32 and shared.shape == (n, d))
     _check(_lib("moe").rllm_moe_combine(_ptr(y), _ptr(place), _ptr(weight), _ptr(out), _ptr(shared), _ptr(gate),
@@ -2010,16 +2082,16 @@ def shared_kv_attention(q, cache, out, ctx, block_table, H, hd, hdv, block_size,
 
 
 def paged_attention(q, k_cache, v_cache, out, ctx, block_table, H, K, hd, block_size, scale, window=0,
-                    keep_first=0, v_head_dim=None, chunk=0, softcap=0.0, sink=None):
+                    keep_first=0, v_head_dim=None, chunk=0, softcap=0.0, sink=None, slopes=None):
     """Attention of the step's tokens over the paged cache; chooses the kernel by element type,
     head size and the shape of the step (`ctx`: the step's StepContext).  float32, head sizes
     other than 64 and 128 and value heads of another size than the key heads take the plain kernel;
     windows that keep the first keys take the mma.sync kernels, not the tcgen05 one."""
     hdv = hd if not v_head_dim else int(v_head_dim)
     keep_first = keep_first if window else 0
-    if q.dtype != torch.bfloat16 or hd not in FLASH_HEAD_DIMS or hdv != hd:
+    if q.dtype != torch.bfloat16 or hd not in FLASH_HEAD_DIMS or hdv != hd or slopes is not None:
         return paged_attention_generic(q, k_cache, v_cache, out, ctx.positions, ctx.seq_ids, block_table,
-                                       H, K, hd, block_size, scale, window, keep_first, hdv, chunk, softcap, sink)
+                                       H, K, hd, block_size, scale, window, keep_first, hdv, chunk, softcap, sink, slopes)
     key = (H // K, window, chunk)
     plan = ctx.plans.get(key)
     if plan is None:

@@ -1,7 +1,7 @@
 // Row-wise helpers that several kinds of layers share; float32 arithmetic whatever the storage
 // type, accurate expf / tanhf / log1pf (no fast-math):
 //
-//   rows_act        out[t, c] = f1(in[t, c] + bias[c]) * f2(mul[t, c / mul_group])   (bias, mul optional;
+//   rows_act        out[t, c] = factor * f1(row_scale[t] * in[t, c] + bias[c]) * f2(mul[t, c / mul_group])   (row_scale, bias, mul optional;
 //                   mul_group > 1: one factor for each run of that many columns, a gate per head)
 //   axpby           out = a * x + b * y                                      (float32)
 //   cat2_cast       out[t] = [x[t] + s * delta[t] | y[t]] in the activation type (delta optional)
@@ -11,22 +11,10 @@
 //                   the paged cache; the value heads may have another size than the key heads, or the
 //                   values are the key columns as projected (v_off = the keys' first column)
 //
-// f1, f2: 0 identity, 1 silu z / (1 + e^-z), 2 relu(z)^2, 3 sigmoid, 4 tanh, 5 softplus.
+// f1, f2: the activations of activations.cuh.
 #include "common.cuh"
-#include <math.h>
+#include "activations.cuh"
 
-enum : int { ACT_NONE = 0, ACT_SILU = 1, ACT_RELU2 = 2, ACT_SIGMOID = 3, ACT_TANH = 4, ACT_SOFTPLUS = 5 };
-
-__device__ __forceinline__ float act_apply(float z, int act) {
-    switch (act) {
-        case ACT_SILU: return z / (1.0f + expf(-z));
-        case ACT_RELU2: { const float r = fmaxf(z, 0.f); return r * r; }
-        case ACT_SIGMOID: return 1.0f / (1.0f + expf(-z));
-        case ACT_TANH: return tanhf(z);
-        case ACT_SOFTPLUS: return z > 20.f ? z : log1pf(expf(z));
-        default: return z;
-    }
-}
 __device__ __forceinline__ float ld_any(const void* p, int dt, size_t i) {
     return dt == RLLM_F32 ? ((const float*)p)[i] : __bfloat162float(((const bf16*)p)[i]);
 }
@@ -37,7 +25,8 @@ __device__ __forceinline__ void st_any(void* p, int dt, size_t i, float v) {
 
 __global__ void rows_act_kernel(const void* in, int in_dt, long long in_stride, const float* __restrict__ bias,
                                 int act1, const void* mul, int mul_dt, long long mul_stride, int act2, void* out,
-                                int out_dt, long long out_stride, int cols, size_t total, int mul_group) {
+                                int out_dt, long long out_stride, int cols, size_t total, int mul_group, float factor,
+                                const float* row_scale) {
     pdl_wait();
     pdl_launch_dependents();
     const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
@@ -45,8 +34,9 @@ __global__ void rows_act_kernel(const void* in, int in_dt, long long in_stride, 
     const size_t t = i / cols;
     const int c = (int)(i - t * cols);
     float v = ld_any(in, in_dt, t * in_stride + c);
+    if (row_scale) v *= row_scale[t];
     if (bias) v += bias[c];
-    v = act_apply(v, act1);
+    v = act_apply(v, act1) * factor;
     if (mul) v *= act_apply(ld_any(mul, mul_dt, t * mul_stride + c / mul_group), act2);
     st_any(out, out_dt, t * out_stride + c, v);
 }
@@ -54,14 +44,14 @@ __global__ void rows_act_kernel(const void* in, int in_dt, long long in_stride, 
 // The gate of an attention's heads on bfloat16 rows: out[t, c] = in[t, c] * f2(mul[t, c / group]) with eight
 // columns (16 bytes) a thread; `group` a multiple of 8, so the eight share a factor.
 __global__ void rows_gate_bf16_kernel(const bf16* in, long long in_stride, const float* mul, long long mul_stride, int act2,
-                                      bf16* out, long long out_stride, int cols8, int group8, size_t total) {
+                                      bf16* out, long long out_stride, int cols8, int group8, size_t total, float factor) {
     pdl_wait();
     pdl_launch_dependents();
     const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
     if (i >= total) return;
     const size_t t = i / cols8;
     const int c8 = (int)(i - t * cols8);
-    const float f = act_apply(mul[t * mul_stride + c8 / group8], act2);
+    const float f = factor * act_apply(mul[t * mul_stride + c8 / group8], act2);
     uint4 u = *reinterpret_cast<const uint4*>(in + t * in_stride + 8 * (size_t)c8);
     __nv_bfloat162* p = reinterpret_cast<__nv_bfloat162*>(&u);
 #pragma unroll
@@ -74,20 +64,21 @@ __global__ void rows_gate_bf16_kernel(const bf16* in, long long in_stride, const
 
 RLLM_API int rllm_rows_act(const void* in, int in_dt, long long in_stride, const float* bias, int act1,
                            const void* mul, int mul_dt, long long mul_stride, int act2, void* out, int out_dt,
-                           long long out_stride, int n, int cols, int mul_group, cudaStream_t stream) {
+                           long long out_stride, int n, int cols, int mul_group, float factor, const float* row_scale,
+                           cudaStream_t stream) {
     const size_t total = (size_t)n * cols;
     if (total == 0) return 0;
     if (mul_group <= 0) return (int)cudaErrorInvalidValue;
     const auto al16 = [](const void* p) { return ((uintptr_t)p & 15) == 0; };
-    if (in_dt == RLLM_BF16 && out_dt == RLLM_BF16 && mul && mul_dt == RLLM_F32 && !bias && act1 == ACT_NONE &&
+    if (in_dt == RLLM_BF16 && out_dt == RLLM_BF16 && mul && mul_dt == RLLM_F32 && !bias && !row_scale && act1 == ACT_NONE &&
         mul_group % 8 == 0 && cols % 8 == 0 && in_stride % 8 == 0 && out_stride % 8 == 0 && al16(in) && al16(out)) {
         const size_t t8 = total / 8;
         return rllm_launch(rows_gate_bf16_kernel, dim3((unsigned)((t8 + 255) / 256)), dim3(256), 0, stream, (const bf16*)in,
-                           in_stride, (const float*)mul, mul_stride, act2, (bf16*)out, out_stride, cols / 8, mul_group / 8, t8);
+                           in_stride, (const float*)mul, mul_stride, act2, (bf16*)out, out_stride, cols / 8, mul_group / 8, t8, factor);
     }
     return rllm_launch(rows_act_kernel, dim3((unsigned)((total + 255) / 256)), dim3(256), 0, stream, in, in_dt,
                        in_stride, bias, act1, mul, mul_dt, mul_stride, act2, out, out_dt, out_stride, cols, total,
-                       mul_group);
+                       mul_group, factor, row_scale);
 }
 
 __global__ void axpby_kernel(float a, const float* x, float b, const float* y, float* out, size_t total) {

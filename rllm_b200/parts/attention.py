@@ -19,6 +19,10 @@ and is not scaled.
 `own_kv` False: the layer has no key and value projections (nor a key norm); it reads the keys (as
 cached: normed and rotated) and values that another layer wrote (the run entry's `cache_of`), with
 queries, sinks and output projection of its own.
+`slopes`: one number per query head (linear position biases): slope_h * (i - j) is taken off the score of the
+query at i and the key at j.
+`cache_window`: the window of keys the cache keeps where it is another one than the layer's own (a layer that
+reads these keys through a longer window; 0: all keys).  Default: `window`.
 `names` "short": the tensors are <prefix>q, k, v, o, q.norm, k.norm, sink.
 """
 from __future__ import annotations
@@ -50,17 +54,21 @@ class Attention(Mixer):
         self.hdv = int(p.get("v_head_dim") or self.hd)
         self.has_sink = bool(p.get("sink", False))
         self.own_kv = bool(p.get("own_kv", True))
+        self.slope_values = tuple(float(x) for x in p["slopes"]) if p.get("slopes") is not None else None
+        if self.slope_values is not None and len(self.slope_values) != self.H:
+            raise PartError(f"attention: {len(self.slope_values)} slopes for {self.H} heads")
+        self.cache_window = int(p["cache_window"] or 0) if "cache_window" in p else self.window
         short = p.get("names") == "short"
-        self.plain = self.hdv == self.hd and not self.has_sink and self.own_kv
-        if (self.hd % 16 and self.plain) or self.hd % 2 or self.hd > 256 or self.hdv > 256:
+        self.plain = self.hdv == self.hd and not self.has_sink and self.own_kv and self.slope_values is None
+        if (self.hd % 16 and self.plain) or (self.hd % 2 and self.slope_values is None) or self.hd > 256 or self.hdv > 256:
             raise PartError(f"attention: head_dim {self.hd} must be a multiple of 16 and at most 256")
         n = (lambda s: s) if short else (lambda s: {"q.norm": "q_norm.weight", "k.norm": "k_norm.weight",
                                                     "sink": "sink"}.get(s, s + "_proj.weight"))
         self._n = {s: self.prefix + n(s) for s in ("q", "k", "v", "o", "q.norm", "k.norm", "sink")}
-        self.w_qkv = self.w_o = self.q_norm_w = self.k_norm_w = self.sink = None
+        self.w_qkv = self.w_o = self.q_norm_w = self.k_norm_w = self.sink = self.slopes = None
 
     def cache_need(self):
-        return PagedKVNeed(self.K, self.hd, self.window, 0, self.hdv if self.hdv != self.hd else 0)
+        return PagedKVNeed(self.K, self.hd, self.cache_window, 0, self.hdv if self.hdv != self.hd else 0)
 
     def expected_tensors(self):
         d, H, K, hd, n = self.hidden_size, self.H, self.K, self.hd, self._n
@@ -86,6 +94,8 @@ class Attention(Mixer):
                 self.k_norm_w = self._to_device(tensors[n["k.norm"]], torch.float32)
         if self.has_sink:
             self.sink = self._to_device(tensors[n["sink"]], torch.float32)
+        if self.slope_values is not None:
+            self.slopes = torch.tensor(self.slope_values, dtype=torch.float64).to(self.runtime.device, torch.float32)
 
     # A norm between two products may go without a kernel of its own (ops.NormedRows): the block asks the
     # parts on both sides for the matrices of their last and first product.
@@ -102,7 +112,7 @@ class Attention(Mixer):
         dt = self.runtime.dtype
         q = torch.empty((n, self.H * self.hd), dtype=dt, device=self.w_qkv.device)
         if not self.plain:
-            return self._forward_general(h, ctx, cache, position, q)
+            return self._forward_general(h, ctx, cache, position, q, residual)
         whole = getattr(position, "project_and_store", None)
         if whole is not None and whole(h, self.w_qkv, self.q_norm_w, self.k_norm_w, self.qk_norm_eps, ctx, cache, q,
                                        self.H, self.K, self.hd):
@@ -130,8 +140,8 @@ class Attention(Mixer):
             return None
         return ops.linear(attn, self.w_o, out_dtype=torch.float32)
 
-    def _forward_general(self, h, ctx, cache, position, q):
-        """Value heads of their own size, sinks, or another layer's keys and values: the position part
+    def _forward_general(self, h, ctx, cache, position, q, residual=None):
+        """Value heads of their own size, sinks, slopes, or another layer's keys and values: the position part
         does norm, rotation and the cache write (`apply_and_store` with `v_head_dim` and `has_kv`)."""
         if cache.write != self.own_kv:
             raise PartError("attention: a layer with keys and values of its own writes its cache; one without "
@@ -146,5 +156,9 @@ class Attention(Mixer):
                                      has_kv=self.own_kv)
         attn = torch.empty((q.shape[0], self.H * self.hdv), dtype=q.dtype, device=q.device)
         ops.paged_attention(q, cache.k, cache.v, attn, ctx, cache.block_table, self.H, self.K, self.hd,
-                            cache.block_size, self.scale, self.window, v_head_dim=self.hdv, sink=self.sink)
+                            cache.block_size, self.scale, self.window, v_head_dim=self.hdv, sink=self.sink,
+                            slopes=self.slopes)
+        if residual is not None:
+            ops.linear(attn, self.w_o, out=residual, accumulate=True)
+            return None
         return ops.linear(attn, self.w_o, out_dtype=torch.float32)

@@ -14,13 +14,16 @@ For normed input rows h [n, d] (H query heads, G key/value heads, key size dk, v
                                                       `gate_per_head` Wg has one row per head and its
                                                       number multiplies the whole head)
 
-With `tie_values` there is no Wv: the values are the key rows as projected, before their norm.
+`qk_norm` "row": an RMS norm over the whole query row and the whole key row, a weight per column; "head": over
+each head, one weight of head_dim entries for all query heads and one for all key heads.  With a position part the heads
+are rotated behind the norm.  With `tie_values` there is no Wv: the values are the key rows as projected, before their norm.
 
-Parameters: hidden_size, num_heads, num_kv_heads, head_dim, v_head_dim, bias, qk_norm ("row" or
+Parameters: hidden_size, num_heads, num_kv_heads, head_dim, v_head_dim, bias, qk_norm ("row", "head" or
 None), eps, window (0: all keys), keep_first, scale, gate ("sigmoid" or None), gate_per_head, tie_values.  Tensors under
 <prefix>: q, k, v, o, g and, by the options, q.b, k.b, v.b, q.norm, k.norm.  Load-time transform:
 q, k, v and the gate are stacked into one projection [q | k | v | g] (the biases of q, k, v likewise; rows of
-zeros up to a multiple of 8 rows).  Scores, softmax, norms and the
+zeros up to a multiple of 8 rows).  ``forward(..., into=, factor=)``: the rows that the output projection
+would read, times `factor`, go to the matrix `into` and the projection is left to the caller (OUTPUT_MATRIX).  Scores, softmax, norms and the
 gate's sigmoid are float32 in every mode.
 """
 from __future__ import annotations
@@ -35,6 +38,7 @@ from .base import Mixer, PagedKVNeed, PartError, register_part
 class GatedWindowAttention(Mixer):
     CAPTURE_SAFE = True
     INPUT_MATRIX = "w_qkv"        # the stacked product on h; a mixer made of mixers may run it with its neighbour's
+    OUTPUT_MATRIX = "w_o"         # and the product behind the heads likewise
 
     def __init__(self, params, prefix, runtime):
         super().__init__(params, prefix, runtime)
@@ -56,8 +60,10 @@ class GatedWindowAttention(Mixer):
             raise PartError("gated_attention: tied values have the keys' head size and no biases")
         if self.H % self.G:
             raise PartError(f"gated_attention: {self.H} heads are not a multiple of {self.G} key/value heads")
-        if self.qk_norm not in (None, "row"):
-            raise PartError(f"gated_attention: qk_norm {self.qk_norm!r} is not supported ('row' or none)")
+        if self.qk_norm not in (None, "row", "head"):
+            raise PartError(f"gated_attention: qk_norm {self.qk_norm!r} is not supported ('row', 'head' or none)")
+        if self.qk_norm == "head" and (self.bias or self.tie_values):
+            raise PartError("gated_attention: a norm per head goes with neither biases nor tied values")
         if self.gate not in (None, "sigmoid", "silu"):
             raise PartError(f"gated_attention: gate {self.gate!r} is not supported")
         if max(self.dk, self.dv) > 512:
@@ -76,7 +82,8 @@ class GatedWindowAttention(Mixer):
         if self.bias:
             t.update({p + "q.b": ((wq,), "bias"), p + "k.b": ((wk,), "bias"), p + "v.b": ((wv,), "bias")})
         if self.qk_norm:
-            t.update({p + "q.norm": ((wq,), "norm"), p + "k.norm": ((wk,), "norm")})
+            nq, nk = (self.dk, self.dk) if self.qk_norm == "head" else (wq, wk)
+            t.update({p + "q.norm": ((nq,), "norm"), p + "k.norm": ((nk,), "norm")})
         if self.gate:
             t[p + "g"] = ((self.H if self.gate_per_head else self.H * self.dv, d), "matrix")
         return t
@@ -97,8 +104,12 @@ class GatedWindowAttention(Mixer):
             self.k_norm_w = self._to_device(tensors[p + "k.norm"], torch.float32)
         self.w_o = self._to_device(tensors[p + "o"])
 
-    def forward(self, h, ctx, cache, position=None, residual=None, rows=None):
-        """`rows`: h . w_qkv^T (float32), where somebody else has run that product."""
+    @property
+    def output_columns(self):
+        return self.H * self.dv
+
+    def forward(self, h, ctx, cache, position=None, residual=None, rows=None, into=None, factor=1.0):
+        """`rows`: h . w_qkv^T (float32), where somebody else has run that product; `into`, `factor`: see above."""
         n, dt, dev = h.shape[0], self.runtime.dtype, h.device
         wide = ops.linear(h, self.w_qkv, out_dtype=torch.float32) if rows is None else rows     # [q | k | v | gate]
         n_qkv = (self.H + self.G) * self.dk + (0 if self.tie_values else self.G * self.dv)
@@ -107,15 +118,24 @@ class GatedWindowAttention(Mixer):
         rot = min(position.dims, self.dk) if position is not None else 0
         if rot and getattr(position, "mult", 1.0) != 1.0:
             raise PartError("gated_attention: cos and sin with a multiplier are not supported")
-        ops.qkv_rownorm_store(qkv, self.b_qkv, self.q_norm_w, self.k_norm_w, cache.slots, q, cache.k, cache.v,
-                              self.H, self.G, self.dk, self.dv, cache.block_size, self.eps, write_kv=cache.write,
-                              cs_table=position.angles(ctx) if rot else None, rot=rot,
-                              pairs=bool(rot) and position.layout == "pairs", v_tied=self.tie_values)
+        if self.qk_norm == "head":
+            ops.head_norm_rope_store(qkv, self.q_norm_w, self.k_norm_w, position.angles(ctx) if rot else None, rot,
+                                     bool(rot) and position.layout == "pairs", cache.slots, q, cache.k, cache.v, self.H,
+                                     self.G, self.dk, self.dv, cache.block_size, self.eps, write_kv=cache.write)
+        else:
+            ops.qkv_rownorm_store(qkv, self.b_qkv, self.q_norm_w, self.k_norm_w, cache.slots, q, cache.k, cache.v,
+                                  self.H, self.G, self.dk, self.dv, cache.block_size, self.eps, write_kv=cache.write,
+                                  cs_table=position.angles(ctx) if rot else None, rot=rot,
+                                  pairs=bool(rot) and position.layout == "pairs", v_tied=self.tie_values)
         attn = torch.empty((n, self.H * self.dv), dtype=dt, device=dev)
         ops.paged_attention(q, cache.k, cache.v, attn, ctx, cache.block_table, self.H, self.G, self.dk,
                             cache.block_size, self.scale, self.window, self.keep_first, self.dv)
         if self.gate:
             n_gate = self.H if self.gate_per_head else self.H * self.dv
-            ops.rows_act(attn, attn, mul=wide[:, n_qkv:n_qkv + n_gate], mul_act=self.gate,
-                         mul_group=self.dv if self.gate_per_head else 1)
+            ops.rows_act(attn, attn if into is None else into, mul=wide[:, n_qkv:n_qkv + n_gate], mul_act=self.gate,
+                         mul_group=self.dv if self.gate_per_head else 1, factor=factor)
+        elif into is not None:
+            ops.rows_act(attn, into, factor=factor)
+        if into is not None:
+            return None
         return ops.linear(attn, self.w_o, out_dtype=torch.float32)

@@ -1,5 +1,5 @@
 """Causal attention through low-rank latents (queries through one, keys and values through another),
-with one rotated key part shared by all heads.
+with one rotated key part shared by all heads, or none (`rot_dim` 0: no positions at all).
 
 For input rows h [n, d] (H heads; per head dq plain and r rotated query/key entries, values of size
 dv; latents of q_rank and kv_rank entries):
@@ -48,8 +48,8 @@ class LatentAttention(Mixer):
         self.scale = float(p["scale"])
         self.softcap = float(p.get("softcap", 0.0) or 0.0)
         self.window = int(p.get("window", 0) or 0)
-        if self.r <= 0 or self.r % 2:
-            raise PartError(f"latent_attention: rot_dim {self.r} must be positive and even")
+        if self.r < 0 or self.r % 2:
+            raise PartError(f"latent_attention: rot_dim {self.r} must be even (0: no rotated part)")
         if self.rank > 512 or self.rank + self.r > 2048:
             raise PartError("latent_attention: kv_rank up to 512, kv_rank + rot_dim up to 2048")
         self.w_down = self.w_uq = self.w_qc = self.w_uv = self.w_o = self.q_norm_w = self.kv_norm_w = None
@@ -84,7 +84,7 @@ class LatentAttention(Mixer):
     def forward(self, h, ctx, cache, position=None, residual=None):
         n, dt, dev = h.shape[0], self.runtime.dtype, h.device
         H, dq, r, rank = self.H, self.dq, self.r, self.rank
-        if position is None or position.dims != r:
+        if (position.dims if position is not None else 0) != r:
             raise PartError("latent_attention: needs a rotary position part over rot_dim entries")
         low = ops.linear(h, self.w_down, out_dtype=torch.float32)              # [query latent | c | kr]
         if self.q_rank:
@@ -96,12 +96,15 @@ class LatentAttention(Mixer):
         W = rank + r
         q_att = torch.empty((n, H * W), dtype=dt, device=dev)
         ops.head_linear(q.view(n, H, dq + r)[:, :, :dq], self.w_qc, q_att.view(n, H, W)[:, :, :rank])
-        ops.latent_rope_store(q, low[:, self.q_rank:], self.kv_norm_w, position.angles(ctx), position.mult,
-                              cache.slots, q_att, cache.k, H, dq, r, rank, cache.block_size, self.eps,
+        ops.latent_rope_store(q, low[:, self.q_rank:], self.kv_norm_w, position.angles(ctx) if r else None,
+                              position.mult if r else 1.0, cache.slots, q_att, cache.k, H, dq, r, rank, cache.block_size, self.eps,
                               write_kv=cache.write, pairs=getattr(position, "layout", "half") == "pairs")
         mixed = torch.empty((n, H * rank), dtype=dt, device=dev)
         ops.shared_kv_attention(q_att, cache.k, mixed, ctx, cache.block_table, H, W, rank, cache.block_size,
                                 self.scale, softcap=self.softcap, window=self.window)
         a = torch.empty((n, H * self.dv), dtype=dt, device=dev)
         ops.head_linear(mixed.view(n, H, rank), self.w_uv, a.view(n, H, self.dv))
+        if residual is not None:
+            ops.linear(a, self.w_o, out=residual, accumulate=True)
+            return None
         return ops.linear(a, self.w_o, out_dtype=torch.float32)

@@ -13,16 +13,18 @@ For normed input rows h [n, d], E experts of size F, each token using `top_k`:
         correction), divided by their sum + `weight_eps` when `normalize`, times `route_scale`
     expert e:  y_e = Wd_e (silu(Wg_e h) * (Wu_e h)), or with `expert_form` = {limit, alpha, shift} the gated unit
                Wd_e (g sigmoid(alpha g) (u + shift)), g = min(Wg_e h, limit), u = clamp(Wu_e h, -limit, limit)
-    out = sum over the chosen e of weight_e * y_e
+               or, with an `activation` f, no gate: Wd_e f(Wu_e h), and the shared one likewise
+    out = sum over the chosen e of weight_e * y_e       (`weigh_input`: the weight multiplies what the expert reads instead,
+                                                          y_e = expert_e(weight_e h), and the sum has no weights)
           + sigmoid(h . w_sg) * shared(h)                (`shared_size` > 0: one more expert of that size
                                                           for every token; `shared_gate`: its gate;
                                                           `shared_form`: its gated form, as above)
 
 Parameters: hidden_size, intermediate_size, num_experts, top_k, n_groups, keep_groups, group_best, score,
-correction, normalize, weight_eps, route_scale, shared_size, shared_gate, router_bias, expert_form, shared_form.  Tensors under <prefix>:
+correction, normalize, weight_eps, route_scale, shared_size, shared_gate, router_bias, expert_form, shared_form, activation, weigh_input.  Tensors under <prefix>:
 router [E, d], router.b [E], correction [E], e<i>.gate, e<i>.up [F, d], e<i>.down [d, F], shared.gate, shared.up,
-shared.down, shared.sg [1, d].  Load-time transform: the experts' matrices are stacked ([E, 2F, d] gate
-rows then up rows, [E, d, F]), and the shared expert's gate row is stacked under the router's so that
+shared.down, shared.sg [1, d] (no gates with an `activation`).  Load-time transform: the experts' matrices are stacked ([E, 2F, d]
+gate rows then up rows, or [E, F, d] up rows, and [E, d, F]), and the shared expert's gate row is stacked under the router's so that
 one product gives both (with rows of zeros up to a multiple of 8 rows).  The router's logits, scores, choice
 and weights are float32 in every mode.
 
@@ -62,6 +64,12 @@ class RoutedExperts(FeedForward):
         self.shared_gate = bool(p.get("shared_gate", False)) and self.shared_size > 0
         form = lambda f: (float(f["limit"]), float(f["alpha"]), float(f["shift"])) if f else None
         self.expert_form, self.shared_form = form(p.get("expert_form")), form(p.get("shared_form"))
+        self.activation, self.weigh_input = p.get("activation"), bool(p.get("weigh_input", False))
+        if self.activation is not None and (self.activation not in ops.ACT or self.expert_form or self.shared_form):
+            raise PartError("routed_experts: an activation by name goes without gated forms")
+        if self.weigh_input and self.activation is None:
+            raise PartError("routed_experts: weights on the experts' inputs need experts without a gate")
+        self.parts_up = ("up",) if self.activation is not None else ("gate", "up")
         if any(f is not None and f[1] == 0.0 for f in (self.expert_form, self.shared_form)):
             raise PartError("routed_experts: a gated form's alpha must not be 0")
         if self.E % self.n_groups or not 0 < self.keep_groups <= self.n_groups:
@@ -80,12 +88,12 @@ class RoutedExperts(FeedForward):
         if self.has_bias:
             t[p + "router.b"] = ((self.E,), "unit")
         for e in range(self.E):
-            t.update({f"{p}e{e}.gate": ((F, d), "matrix"), f"{p}e{e}.up": ((F, d), "matrix"),
-                      f"{p}e{e}.down": ((d, F), "matrix")})
+            t.update({f"{p}e{e}.{s}": ((F, d), "matrix") for s in self.parts_up})
+            t[f"{p}e{e}.down"] = ((d, F), "matrix")
         if self.shared_size:
             S = self.shared_size
-            t.update({p + "shared.gate": ((S, d), "matrix"), p + "shared.up": ((S, d), "matrix"),
-                      p + "shared.down": ((d, S), "matrix")})
+            t.update({f"{p}shared.{s}": ((S, d), "matrix") for s in self.parts_up})
+            t[p + "shared.down"] = ((d, S), "matrix")
             if self.shared_gate:
                 t[p + "shared.sg"] = ((1, d), "matrix")
         return t
@@ -104,11 +112,10 @@ class RoutedExperts(FeedForward):
         if self.has_bias:
             self.router_bias = self._to_device(tensors[p + "router.b"], torch.float32)
         self.w_gu = self._to_device(torch.stack(
-            [torch.cat([tensors[f"{p}e{e}.gate"].to(dt), tensors[f"{p}e{e}.up"].to(dt)], 0) for e in range(self.E)], 0))
+            [torch.cat([tensors[f"{p}e{e}.{s}"].to(dt) for s in self.parts_up], 0) for e in range(self.E)], 0))
         self.w_down = self._to_device(torch.stack([tensors[f"{p}e{e}.down"].to(dt) for e in range(self.E)], 0))
         if self.shared_size:
-            self.w_shared_gu = self._to_device(torch.cat([tensors[p + "shared.gate"].to(dt),
-                                                          tensors[p + "shared.up"].to(dt)], 0))
+            self.w_shared_gu = self._to_device(torch.cat([tensors[f"{p}shared.{s}"].to(dt) for s in self.parts_up], 0))
             self.w_shared_down = self._to_device(tensors[p + "shared.down"])
 
     def route(self, h):
@@ -127,24 +134,41 @@ class RoutedExperts(FeedForward):
         shared = gate = None
         if self.shared_size:
             act = torch.empty((n, self.shared_size), dtype=dt, device=dev)
-            ops.gate_up_swiglu(h, self.w_shared_gu, act, glu=self.shared_form)
+            if self.activation is not None:
+                ops.rows_act(ops.linear(h, self.w_shared_gu, out_dtype=torch.float32), act, act=self.activation)
+            else:
+                ops.gate_up_swiglu(h, self.w_shared_gu, act, glu=self.shared_form)
             shared = ops.linear(act, self.w_shared_down, out_dtype=torch.float32)
             gate = logits[:, self.E:self.E + 1] if self.shared_gate else None
         out = torch.empty((n, d), dtype=torch.float32, device=dev)
         if n <= PAIR_ROWS or torch.cuda.is_current_stream_capturing():
             act = torch.empty((n * self.top_k, self.F), dtype=dt, device=dev)
-            ops.moe_pairs_gate_up(h, self.w_gu, idx, act, glu=self.expert_form or (0.0, 1.0, 0.0))
+            if self.activation is not None:
+                ops.moe_pairs_up(h, self.w_gu, idx, weight if self.weigh_input else None, act, self.activation)
+            else:
+                ops.moe_pairs_gate_up(h, self.w_gu, idx, act, glu=self.expert_form or (0.0, 1.0, 0.0))
+            if self.weigh_input:
+                weight = None                              # the experts' inputs have had it
             return ops.moe_pairs_down(act, self.w_down, idx, weight, out, shared, gate)
         # many rows: the pairs in expert order, each expert's rows through the package's products
         offsets, place = ops.moe_sort(idx, self.E)
         rows = torch.empty((n * self.top_k, d), dtype=dt, device=dev)
-        ops.moe_gather_rows(h, place, rows, self.top_k)
+        w_rows = torch.empty(n * self.top_k, dtype=torch.float32, device=dev) if self.weigh_input else None
+        ops.moe_gather_rows(h, place, rows, self.top_k, weight if self.weigh_input else None, w_rows)
         bounds = offsets.tolist()                          # the host learns how many rows each expert has
         act = torch.empty((n * self.top_k, self.F), dtype=dt, device=dev)
         y = torch.empty((n * self.top_k, d), dtype=torch.float32, device=dev)
+        if self.activation is not None:
+            up = torch.empty((n * self.top_k, self.F), dtype=torch.float32, device=dev)
+            for e in range(self.E):
+                a, b = bounds[e], bounds[e + 1]
+                if b > a:
+                    ops.linear(rows[a:b], self.w_gu[e], out=up[a:b])
+            ops.rows_act(up, act, act=self.activation, row_scale=w_rows)
         for e in range(self.E):
             a, b = bounds[e], bounds[e + 1]
-            if b > a:
+            if b > a and self.activation is None:
                 ops.gate_up_swiglu(rows[a:b], self.w_gu[e], act[a:b], glu=self.expert_form)
+            if b > a:
                 ops.linear(act[a:b], self.w_down[e], out=y[a:b])
-        return ops.moe_combine(y, place, weight, out, shared, gate)
+        return ops.moe_combine(y, place, None if self.weigh_input else weight, out, shared, gate, self.top_k)
