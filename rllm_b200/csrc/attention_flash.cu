@@ -51,7 +51,13 @@ struct FlashParams {
                               // cap_out = cap * log2(e)
     const float* sink;        // [H] or null: exp(sink[h]) joins the denominator of head h's softmax (no key, no value,
                               // not scaled); added once, where a row is normalized
+    const float* slopes;      // [H] or null: slopes[h] * (position - key) is taken off head h's scores
 };
+
+// a head's slope in base-2 exponents (0: none)
+__device__ __forceinline__ float flash_slope(const FlashParams& p, int head) {
+    return p.slopes ? p.slopes[head] * 1.4426950408889634f : 0.f;
+}
 
 // what a head's sink adds to a row's denominator whose running maximum (base 2) is m
 __device__ __forceinline__ float flash_sink_term(const FlashParams& p, int head, float m) {
@@ -156,6 +162,7 @@ __global__ void __launch_bounds__(NW * 32) paged_flash_attention_kernel(const Fl
         if (pos1 >= 0) first1 = max(first1, pos1 - pos1 % p.chunk);
     }
     const int hi0 = min(pos0 + 1, ke), hi1 = min(pos1 + 1, ke);
+    const float sl0 = flash_slope(p, head0 + (valid0 ? hl0 : 0)), sl1 = flash_slope(p, head0 + (valid1 ? hl1 : 0));
 
     if (kb >= ke) {                                // an empty split: mark it so
         if (p.split_keys > 0 && t == 0) {
@@ -261,8 +268,9 @@ __global__ void __launch_bounds__(NW * 32) paged_flash_attention_kernel(const Fl
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
                 float v = flash_exponent(p, s[j][e]);
+                const int key = kt + 8 * j + 2 * t + (e & 1);
+                if (p.slopes) v = fmaf(e < 2 ? sl0 : sl1, (float)(key - (e < 2 ? pos0 : pos1)), v);
                 if (need_mask) {
-                    const int key = kt + 8 * j + 2 * t + (e & 1);
                     const bool vis = (e < 2) ? ((key >= f0 || key < keepv) && key < h0)
                                              : ((key >= f1 || key < keepv) && key < h1);
                     if (!vis) v = -INFINITY;
@@ -408,7 +416,8 @@ __global__ void __launch_bounds__(32) paged_decode_attention_kernel(const FlashP
     const size_t part_base = (((size_t)tile * gridDim.y + blockIdx.y) * gridDim.z + blockIdx.z) * p.part_rows;
 
     // the two columns (query rows) of this lane's accumulators: 2t and 2t + 1
-    int rowc[2], tlc[2], hlc[2], firstc[2], hic[2];
+    int rowc[2], tlc[2], hlc[2], firstc[2], hic[2], posc[2];
+    float slc[2];
     bool validc[2];
 #pragma unroll
     for (int x = 0; x < 2; ++x) {
@@ -420,6 +429,8 @@ __global__ void __launch_bounds__(32) paged_decode_attention_kernel(const FlashP
         firstc[x] = (p.window > 0 && !sink_split) ? max(0, pos + 1 - p.window) : 0;
         if (p.chunk > 0 && pos >= 0) firstc[x] = max(firstc[x], pos - pos % p.chunk);
         hic[x] = min(pos + 1, ke);
+        posc[x] = pos;
+        slc[x] = flash_slope(p, head0 + (validc[x] ? hlc[x] : 0));
     }
     if (kb >= ke) {                                // an empty split: mark it so
         pdl_wait();                                // the partials of the layer before may still be read
@@ -569,9 +580,9 @@ __global__ void __launch_bounds__(32) paged_decode_attention_kernel(const FlashP
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
                 float v = flash_exponent(p, s[j][e]);
+                const int key = kt + 16 * j + g + (e >> 1) * 8, x = e & 1;
+                if (p.slopes) v = fmaf(slc[x], (float)(key - posc[x]), v);
                 if (need_mask) {
-                    const int key = kt + 16 * j + g + (e >> 1) * 8;
-                    const int x = e & 1;
                     if (!((key >= firstc[x] || key < keepv) && key < hic[x])) v = -INFINITY;
                 }
                 s[j][e] = v;
@@ -757,13 +768,15 @@ static int launch_flash(const FlashParams& p, int mode, int n_tiles, int n_split
 // chunk > 0: the chunked mask (runs of `chunk` positions counted from 0; a token sees the keys of its
 // own run up to itself).  softcap > 0: scores go through softcap * tanh(s * scale / softcap).
 // sink (one float per query head, or null): exp(sink[h]) joins the softmax's denominator of head h.
-RLLM_API int rllm_paged_flash_attention_sink(const void* q, const void* k_cache, const void* v_cache, void* out,
+// slopes (one float per query head, or null): slopes[h] * (i - j) is taken off the score of the query at i and the key at j
+// (behind the cap).
+RLLM_API int rllm_paged_flash_attention_sloped(const void* q, const void* k_cache, const void* v_cache, void* out,
                                              float* part_o, float* part_ml, const int* positions, const int* cu_q,
                                              const int* block_table, int table_stride, const int* tile_req,
                                              const int* tile_tok0, int n_tiles, int H, int K, int hd, int bs,
                                              float scale, int window, int keep_first, int mode, int TT, int GH,
                                              int head_chunks, int split_keys, int n_splits, long long n_pages,
-                                             int* err, int chunk, float softcap, const float* sink,
+                                             int* err, int chunk, float softcap, const float* sink, const float* slopes,
                                              cudaStream_t stream) {
     if (n_tiles <= 0) return 0;
     if (chunk < 0 || softcap < 0.f) return (int)cudaErrorInvalidValue;
@@ -786,9 +799,24 @@ RLLM_API int rllm_paged_flash_attention_sink(const void* q, const void* k_cache,
     p.cap_in = softcap > 0.f ? scale / softcap : 0.f;
     p.cap_out = softcap > 0.f ? softcap * 1.4426950408889634f : 0.f;
     p.sink = sink;
+    p.slopes = slopes;
     if (hd == 128) return launch_flash<128>(p, mode, n_tiles, n_splits, stream);
     if (hd == 64) return launch_flash<64>(p, mode, n_tiles, n_splits, stream);
     return (int)cudaErrorInvalidValue;
+}
+
+RLLM_API int rllm_paged_flash_attention_sink(const void* q, const void* k_cache, const void* v_cache, void* out,
+                                             float* part_o, float* part_ml, const int* positions, const int* cu_q,
+                                             const int* block_table, int table_stride, const int* tile_req,
+                                             const int* tile_tok0, int n_tiles, int H, int K, int hd, int bs,
+                                             float scale, int window, int keep_first, int mode, int TT, int GH,
+                                             int head_chunks, int split_keys, int n_splits, long long n_pages,
+                                             int* err, int chunk, float softcap, const float* sink,
+                                             cudaStream_t stream) {
+    return rllm_paged_flash_attention_sloped(q, k_cache, v_cache, out, part_o, part_ml, positions, cu_q, block_table,
+                                             table_stride, tile_req, tile_tok0, n_tiles, H, K, hd, bs, scale, window,
+                                             keep_first, mode, TT, GH, head_chunks, split_keys, n_splits, n_pages, err,
+                                             chunk, softcap, sink, nullptr, stream);
 }
 
 RLLM_API int rllm_paged_flash_attention_masked(const void* q, const void* k_cache, const void* v_cache, void* out,
@@ -889,3 +917,4 @@ RLLM_PACKED(rllm_paged_flash_attention)
 RLLM_PACKED(rllm_paged_flash_attention_kept)
 RLLM_PACKED(rllm_paged_flash_attention_masked)
 RLLM_PACKED(rllm_paged_flash_attention_sink)
+RLLM_PACKED(rllm_paged_flash_attention_sloped)

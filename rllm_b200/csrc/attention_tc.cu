@@ -73,6 +73,8 @@ struct AttnTcParams {
                                 // cap_in = scale / cap and cap_pre = cap / scale
     const float* sink;          // [H] or null: exp(sink[h]) joins the denominator of head h's softmax (no key, no value,
                                 // not scaled); added once, where a row is normalized
+    const float* slopes;        // [H] or null: slopes[h] * (position - key) is taken off head h's scores
+    float inv_scale;            // 1 / scale: the slopes are applied to the raw scores
 };
 
 // K-major, 128-byte swizzle (Q, K, P): see smem_desc_sw128.  MN-major (V: dims contiguous):
@@ -306,6 +308,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
         const int pos_r = valid ? p.positions[tok0 + tl] : -1;
         int first_r = p.window > 0 ? max(0, pos_r + 1 - p.window) : 0;
         if (p.chunk > 0 && pos_r >= 0) first_r = max(first_r, pos_r - pos_r % p.chunk);
+        const float slope_raw = p.slopes ? p.slopes[head0 + (valid ? hl : 0)] * p.inv_scale : 0.f;
         const int bar_mine = 1 + wg * 4 + quarter;           // arrived at by this warp, waited for by its partner
         const int bar_partner = 1 + (1 - wg) * 4 + quarter;
         const int b = wg;
@@ -340,6 +343,11 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
 #pragma unroll
                     for (int c = 0; c < AT_BN; ++c)
                         sv[c] = p.cap_pre * (1.0f - __fdividef(2.0f, ex2_approx(sv[c] * two_in_log2) + 1.0f));
+                }
+                if (p.slopes) {
+                    const float far = (float)(kt - pos_r);                       // distances are whole numbers: exact
+#pragma unroll
+                    for (int c = 0; c < AT_BN; ++c) sv[c] = fmaf(slope_raw, far + (float)c, sv[c]);
                 }
                 // The maximum is taken over the raw scores (the scale is positive) and the scale goes
                 // into the exponent's multiply-add: one FFMA and one MUFU per score.
@@ -492,11 +500,13 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
 // Returns cudaErrorInvalidValue for shapes outside the limits named at the top of this file.
 // chunk > 0: the chunked mask; softcap > 0: scores go through softcap * tanh(s * scale / softcap).
 // sink (one float per query head, or null): exp(sink[h]) joins the softmax's denominator of head h.
-RLLM_API int rllm_attention_tc_sink(const void* q, const void* k_cache, const void* v_cache, void* out, int n_tokens,
+// slopes (one float per query head, or null): slopes[h] * (i - j) is taken off the score of the query at i and the key at j
+// (behind the cap).
+RLLM_API int rllm_attention_tc_sloped(const void* q, const void* k_cache, const void* v_cache, void* out, int n_tokens,
                                     long long n_pages, const int* positions, const int* cu_q, const int* block_table,
                                     int table_stride, const int* tile_req, const int* tile_tok0, int n_tiles, int H,
                                     int K, int hd, int bs, float scale, int window, int chunk, float softcap,
-                                    const float* sink, int* err, cudaStream_t stream) {
+                                    const float* sink, const float* slopes, int* err, cudaStream_t stream) {
     if (n_tiles <= 0) return 0;
     if (chunk < 0 || softcap < 0.f || !(scale > 0.f)) return (int)cudaErrorInvalidValue;
     if (hd != AT_HD || K <= 0 || H % K || bs < 8 || bs > 128 || (bs & (bs - 1)) || !err) return (int)cudaErrorInvalidValue;
@@ -531,6 +541,8 @@ RLLM_API int rllm_attention_tc_sink(const void* q, const void* k_cache, const vo
     p.cap_in = softcap > 0.f ? scale / softcap : 0.f;
     p.cap_pre = softcap > 0.f ? softcap / scale : 0.f;
     p.sink = sink;
+    p.slopes = slopes;
+    p.inv_scale = 1.0f / scale;
     constexpr int smem = (1 + AT_KS + AT_VS) * AT_TILE_BYTES + 1024;
     static bool attr_set = false;
     if (!attr_set) {
@@ -539,6 +551,16 @@ RLLM_API int rllm_attention_tc_sink(const void* q, const void* k_cache, const vo
         attr_set = true;
     }
     return rllm_launch(attention_tc_kernel, dim3(n_tiles, K), dim3(AT_THREADS), smem, stream, tq, tk, tv, p);
+}
+
+RLLM_API int rllm_attention_tc_sink(const void* q, const void* k_cache, const void* v_cache, void* out, int n_tokens,
+                                    long long n_pages, const int* positions, const int* cu_q, const int* block_table,
+                                    int table_stride, const int* tile_req, const int* tile_tok0, int n_tiles, int H,
+                                    int K, int hd, int bs, float scale, int window, int chunk, float softcap,
+                                    const float* sink, int* err, cudaStream_t stream) {
+    return rllm_attention_tc_sloped(q, k_cache, v_cache, out, n_tokens, n_pages, positions, cu_q, block_table, table_stride,
+                                    tile_req, tile_tok0, n_tiles, H, K, hd, bs, scale, window, chunk, softcap, sink, nullptr, err,
+                                    stream);
 }
 
 RLLM_API int rllm_attention_tc_masked(const void* q, const void* k_cache, const void* v_cache, void* out, int n_tokens,
@@ -566,3 +588,4 @@ TC_DEFINE_WAIT_CONTROLS(rllm_attn_tc)
 RLLM_PACKED(rllm_attention_tc)
 RLLM_PACKED(rllm_attention_tc_masked)
 RLLM_PACKED(rllm_attention_tc_sink)
+RLLM_PACKED(rllm_attention_tc_sloped)

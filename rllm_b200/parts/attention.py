@@ -21,6 +21,9 @@ cached: normed and rotated) and values that another layer wrote (the run entry's
 queries, sinks and output projection of its own.
 `slopes`: one number per query head (linear position biases): slope_h * (i - j) is taken off the score of the
 query at i and the key at j.
+In bfloat16, sloped heads without a norm and of sizes that the tensor-core attention kernels do not take (up to 128
+entries) are stored with zeros behind them up to the next size that they do (rows of zeros in the stacked projection, columns
+of zeros in the output projection), so that those kernels run.
 `cache_window`: the window of keys the cache keeps where it is another one than the layer's own (a layer that
 reads these keys through a longer window; 0: all keys).  Default: `window`.
 `names` "short": the tensors are <prefix>q, k, v, o, q.norm, k.norm, sink.
@@ -58,6 +61,12 @@ class Attention(Mixer):
         if self.slope_values is not None and len(self.slope_values) != self.H:
             raise PartError(f"attention: {len(self.slope_values)} slopes for {self.H} heads")
         self.cache_window = int(p["cache_window"] or 0) if "cache_window" in p else self.window
+        # the sizes heads are stored with: hd, hdv, or both rounded up to a size of the tensor-core kernels
+        self.hd_s, self.hdv_s = self.hd, self.hdv
+        if not runtime.is_f32 and not self.qk_norm and self.slope_values is not None:
+            size = next((s for s in sorted(ops.FLASH_HEAD_DIMS) if max(self.hd, self.hdv) <= s), 0)
+            if size:
+                self.hd_s = self.hdv_s = size
         short = p.get("names") == "short"
         self.plain = self.hdv == self.hd and not self.has_sink and self.own_kv and self.slope_values is None
         if (self.hd % 16 and self.plain) or (self.hd % 2 and self.slope_values is None) or self.hd > 256 or self.hdv > 256:
@@ -68,7 +77,7 @@ class Attention(Mixer):
         self.w_qkv = self.w_o = self.q_norm_w = self.k_norm_w = self.sink = self.slopes = None
 
     def cache_need(self):
-        return PagedKVNeed(self.K, self.hd, self.cache_window, 0, self.hdv if self.hdv != self.hd else 0)
+        return PagedKVNeed(self.K, self.hd_s, self.cache_window, 0, self.hdv_s if self.hdv_s != self.hd_s else 0)
 
     def expected_tensors(self):
         d, H, K, hd, n = self.hidden_size, self.H, self.K, self.hd, self._n
@@ -86,8 +95,17 @@ class Attention(Mixer):
 
     def load(self, tensors):
         n, dt = self._n, self.runtime.dtype
-        self.w_qkv = self._to_device(torch.cat([tensors[n[s]].to(dt) for s in ("qkv" if self.own_kv else "q")], 0))
-        self.w_o = self._to_device(tensors[n["o"]])
+        def stored(t, heads, size, to):              # [heads * size, d] -> [heads * to, d], zeros behind every head
+            if to == size:
+                return t
+            out = t.new_zeros((heads, to, t.shape[1]))
+            out[:, :size] = t.view(heads, size, t.shape[1])
+            return out.view(heads * to, t.shape[1])
+        sizes = {"q": (self.H, self.hd, self.hd_s), "k": (self.K, self.hd, self.hd_s), "v": (self.K, self.hdv, self.hdv_s)}
+        self.w_qkv = self._to_device(torch.cat([stored(tensors[n[s]].to(dt), *sizes[s])
+                                                for s in ("qkv" if self.own_kv else "q")], 0))
+        self.w_o = self._to_device(stored(tensors[n["o"]].t().contiguous(), self.H, self.hdv, self.hdv_s).t()
+                                   if self.hdv_s != self.hdv else tensors[n["o"]])
         if self.qk_norm:
             self.q_norm_w = self._to_device(tensors[n["q.norm"]], torch.float32)
             if self.own_kv:
@@ -110,7 +128,7 @@ class Attention(Mixer):
         norm that follows and the rows come back as ops.NormedRows (needs `residual`)."""
         n = h.shape[0]
         dt = self.runtime.dtype
-        q = torch.empty((n, self.H * self.hd), dtype=dt, device=self.w_qkv.device)
+        q = torch.empty((n, self.H * self.hd_s), dtype=dt, device=self.w_qkv.device)
         if not self.plain:
             return self._forward_general(h, ctx, cache, position, q, residual)
         whole = getattr(position, "project_and_store", None)
@@ -149,14 +167,14 @@ class Attention(Mixer):
         qkv = ops.linear(h, self.w_qkv, out_dtype=torch.float32)              # [q (| k | v)]
         if position is not None:
             position.apply_and_store(qkv, self.q_norm_w, self.k_norm_w, self.qk_norm_eps, ctx, cache, q,
-                                     self.H, self.K, self.hd, v_head_dim=self.hdv, has_kv=self.own_kv)
+                                     self.H, self.K, self.hd_s, v_head_dim=self.hdv_s, has_kv=self.own_kv)
         else:
             ops.head_norm_rope_store(qkv, self.q_norm_w, self.k_norm_w, None, 0, False, cache.slots, q, cache.k,
-                                     cache.v, self.H, self.K, self.hd, self.hdv, cache.block_size, self.qk_norm_eps,
+                                     cache.v, self.H, self.K, self.hd_s, self.hdv_s, cache.block_size, self.qk_norm_eps,
                                      has_kv=self.own_kv)
-        attn = torch.empty((q.shape[0], self.H * self.hdv), dtype=q.dtype, device=q.device)
-        ops.paged_attention(q, cache.k, cache.v, attn, ctx, cache.block_table, self.H, self.K, self.hd,
-                            cache.block_size, self.scale, self.window, v_head_dim=self.hdv, sink=self.sink,
+        attn = torch.empty((q.shape[0], self.H * self.hdv_s), dtype=q.dtype, device=q.device)
+        ops.paged_attention(q, cache.k, cache.v, attn, ctx, cache.block_table, self.H, self.K, self.hd_s,
+                            cache.block_size, self.scale, self.window, v_head_dim=self.hdv_s, sink=self.sink,
                             slopes=self.slopes)
         if residual is not None:
             ops.linear(attn, self.w_o, out=residual, accumulate=True)
