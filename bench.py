@@ -215,10 +215,29 @@ def rusolorn_shape(width: int) -> dict:
             "embedding": {"scale": 8.0}, "residual_mult": 0.5, "token_side": {"dim": 256}}
 
 
+def pibavik_shape(width: int) -> dict:
+    """A Pibavik configuration with layer sizes of a real model of that width: windowed attention with score slopes (width/128
+    heads of 128, a quarter as many key/value heads, a window of 1,024 keys), the same on the first layer's keys and values,
+    attention through latents of 512 entries (heads of 128, queries through 3/8 width, at most 1,536), two layers of windowed
+    attention (half of each head rotated, a norm per head, a gate per head) beside Mamba-2 (inner size 2 widths, heads of 64,
+    128 state entries, 8 groups, 4 taps), attention through latents again: six layers, each with 16 experts of 3/8 width of which
+    a token uses 4 and a shared one of 3/4 width."""
+    heads = max(8, width // 128)
+    att = {"heads": heads, "kv_heads": max(1, heads // 4), "dim": 128, "vdim": 128, "mask": {"size": 1024}, "scale": 128 ** -0.5}
+    latent = {"heads": heads, "dim": 128, "vdim": 128, "kv_rank": 512, "q_rank": min(1536, 3 * width // 8), "scale": 128 ** -0.5}
+    par = {"left": dict(att, rot={"dims": 64, "base": 500000.0}), "left_scale": 0.6, "right_scale": 0.8,
+           "right": {"heads": 2 * width // 64, "vdim": 64, "state": 128, "groups": 8, "conv": 4, "norm_groups": 8}}
+    moe = {"kind": "moe", "expert": {"ff": 3 * width // 8}, "shared": {"ff": 3 * width // 4}, "router": {"experts": 16, "top": 4}}
+    layers = [("attention", att), ("attention", dict(att, kv_from=0)), ("latent_attention", latent), ("parallel", par),
+              ("parallel", par), ("latent_attention", latent)]
+    return {"architecture": "Pibavik", "vocab": 32768, "width": width, "embedding": {"scale": 8.0}, "norm": {"eps": 1e-6},
+            "layers": [{"type": t, "mixer": m, "mlp": moe} for t, m in layers]}
+
+
 FAMILY_SHAPES = {"falalix": falalix_shape, "govopel": govopel_shape, "divuzen": divuzen_shape, "navulorn": navulorn_shape,
-                 "rusolorn": rusolorn_shape}
+                 "rusolorn": rusolorn_shape, "pibavik": pibavik_shape}
 # the model a family stands beside: Qwen3-shaped of equal width, depth and feed-forward, unless another family is closer
-BESIDE = {"navulorn": "divuzen", "rusolorn": "divuzen"}
+BESIDE = {"navulorn": "divuzen", "rusolorn": "divuzen", "pibavik": "rusolorn"}
 
 
 def falalix_compare(a):
@@ -330,15 +349,16 @@ def main():
     ap.add_argument("--ctx", type=int, default=None, help="tokens a request may hold (default: twice the prompt)")
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--skip-points", action="store_true", help="leave out batch 1 / 64 and prefill")
-    ap.add_argument("--workload", default="decode", choices=["decode", "serving", "falalix", "govopel", "divuzen", "navulorn", "rusolorn"],
+    ap.add_argument("--workload", default="decode", choices=["decode", "serving", "falalix", "govopel", "divuzen", "navulorn", "rusolorn", "pibavik"],
                     help="decode: the default line.  serving: --requests prompts of 16..2,048 tokens with 128..512 "
                          "generated tokens each through LLM.generate (continuous batching), one line of its own.  "
                          "falalix: prefill and decode of Falalix-shaped models (--sizes) beside Qwen3-shaped models of "
                          "equal width, depth and feed-forward, one line of its own.  govopel, divuzen: the same for "
                          "Govopel-shaped and for Divuzen-shaped models.  navulorn: Navulorn-shaped beside Divuzen-shaped "
                          "models of equal width and depth.  rusolorn: Rusolorn-shaped beside Divuzen-shaped models "
-                         "of equal width and about equal weights (six layers of two mixers each beside eight of one)")
-    ap.add_argument("--sizes", default="1k,2k,4k", help="falalix, govopel, divuzen, navulorn, rusolorn: model widths to run (1k, 2k, 4k)")
+                         "of equal width and about equal weights (six layers of two mixers each beside eight of one).  "
+                         "pibavik: Pibavik-shaped beside Rusolorn-shaped models of equal width, depth and experts")
+    ap.add_argument("--sizes", default="1k,2k,4k", help="falalix, govopel, divuzen, navulorn, rusolorn, pibavik: model widths to run (1k, 2k, 4k)")
     ap.add_argument("--requests", type=int, default=64)
     ap.add_argument("--parallel", type=int, default=32, help="serving: requests running at once")
     ap.add_argument("--prefill-chunk", type=int, default=512, help="serving: prompt tokens per step")

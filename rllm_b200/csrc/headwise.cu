@@ -10,9 +10,11 @@
 //                      square; queries out, keys into the paged cache; the values written beside them
 //                      are the key heads as projected (before rotation and norm), or the columns that
 //                      follow the keys when the row has them.
-//   latent_rope_store  one cache row per token [normed latent (rank) | rotated shared key part (r, or none)],
+//   latent_rope_store  one cache row per token [normed latent (rank) | rotated shared key part (r)],
 //                      and the rotated part of every query head copied behind that head's latent-space
 //                      query.
+//   latent_norm_store  the same step without rotated parts: both latents of a token normed in one kernel, the query's out in
+//                      the activation type, the other into its cache row (zeros behind it up to the row's length).
 //   head_norm_rope_store  per head of a [q | k | v] projection row: RMS norm with a weight, then the
 //                      rotation of the first `rot` entries (either pair layout); queries out, keys and
 //                      values (heads of another size) into the paged cache; rows of queries only too.
@@ -271,7 +273,7 @@ RLLM_API int rllm_latent_rope_store(const void* q, int q_dt, long long ld_q, con
                                     int bs, float eps, int write_kv, long long n_slots, int* err, int pairs,
                                     cudaStream_t stream) {
     if (n <= 0) return 0;
-    if (H <= 0 || dq <= 0 || r < 0 || (r & 1) || rank <= 0 || bs <= 0 || (r && !cs_table) || !kv_norm_w ||
+    if (H <= 0 || dq <= 0 || r <= 0 || (r & 1) || rank <= 0 || bs <= 0 || !cs_table || !kv_norm_w ||
         ld_q < (long long)H * (dq + r) || ld_kv < rank + r)
         return (int)cudaErrorInvalidValue;
     const int ns = (int)(n_slots > 0x7fffffffLL ? 0x7fffffffLL : n_slots);
@@ -284,6 +286,56 @@ RLLM_API int rllm_latent_rope_store(const void* q, int q_dt, long long ld_q, con
     if (q_dt == RLLM_BF16 && out_dt == RLLM_BF16) { LAUNCH(bf16, bf16); }
     return (int)cudaErrorInvalidValue;
 #undef LAUNCH
+}
+
+// One block per token and latent.  low[t] = [query latent (q_rank, may be 0) | latent (rank)] in float32; each divided by its root
+// mean square and multiplied by its weight; the first to cq [n, q_rank], the second to the token's cache row of W >= rank entries.
+template <typename TO>
+__global__ void __launch_bounds__(256)
+latent_norm_store_kernel(const float* low, long long ld, const float* __restrict__ q_w, const float* __restrict__ kv_w,
+                         const int* __restrict__ slots, TO* cq, TO* cache, int q_rank, int rank, int W, float eps, int write_kv,
+                         int n_slots, int* err) {
+    __shared__ float red[33];
+    pdl_launch_dependents();
+    pdl_wait();
+    const int t = blockIdx.x, tid = threadIdx.x;
+    const float *rq = low + (size_t)t * ld, *rk = rq + q_rank;
+    if (blockIdx.y == 0 && q_rank > 0) {
+        float ss = 0.f;
+        for (int i = tid; i < q_rank; i += blockDim.x) ss += rq[i] * rq[i];
+        ss = block_sum(ss, red);
+        const float rs = 1.0f / sqrtf(ss / (float)q_rank + eps);
+        for (int i = tid; i < q_rank; i += blockDim.x) cq[(size_t)t * q_rank + i] = from_f<TO>(rq[i] * rs * q_w[i]);
+        return;
+    }
+    if (!write_kv) return;
+    float ss = 0.f;
+    for (int i = tid; i < rank; i += blockDim.x) ss += rk[i] * rk[i];
+    ss = block_sum(ss, red);
+    int slot = slots[t];
+    if (slot >= n_slots) {
+        if (tid == 0 && err) atomicExch(err, RLLM_ERR_SLOT);
+        slot = -1;
+    }
+    if (slot < 0) return;
+    const float rs = 1.0f / sqrtf(ss / (float)rank + eps);
+    TO* dst = cache + (size_t)slot * W;
+    for (int i = tid; i < W; i += blockDim.x) dst[i] = from_f<TO>(i < rank ? rk[i] * rs * kv_w[i] : 0.f);
+}
+
+RLLM_API int rllm_latent_norm_store(const float* low, long long ld, const float* q_w, const float* kv_w, const int* slots, void* cq,
+                                    void* cache, int out_dt, int n, int q_rank, int rank, int W, float eps, int write_kv,
+                                    long long n_slots, int* err, cudaStream_t stream) {
+    if (n <= 0) return 0;
+    if (q_rank < 0 || rank <= 0 || W < rank || ld < q_rank + rank || (q_rank > 0 && (!q_w || !cq)) || !kv_w)
+        return (int)cudaErrorInvalidValue;
+    const int ns = (int)(n_slots > 0x7fffffffLL ? 0x7fffffffLL : n_slots);
+    const dim3 grid(n, q_rank > 0 ? 2 : 1);
+    if (out_dt == RLLM_F32)
+        return rllm_launch(latent_norm_store_kernel<float>, grid, dim3(256), 0, stream, low, ld, q_w, kv_w, slots, (float*)cq,
+                           (float*)cache, q_rank, rank, W, eps, write_kv, ns, err);
+    return rllm_launch(latent_norm_store_kernel<bf16>, grid, dim3(256), 0, stream, low, ld, q_w, kv_w, slots, (bf16*)cq,
+                       (bf16*)cache, q_rank, rank, W, eps, write_kv, ns, err);
 }
 
 // ------------------------------------------------------------------ norm after the residual sum
@@ -737,6 +789,7 @@ RLLM_PACKED(rllm_masked_softmax_rows)
 RLLM_PACKED(rllm_norm_rows)
 RLLM_PACKED(rllm_rope_unitnorm_store)
 RLLM_PACKED(rllm_latent_rope_store)
+RLLM_PACKED(rllm_latent_norm_store)
 RLLM_PACKED(rllm_glu_clamped)
 RLLM_PACKED(rllm_sum_norm_rows)
 RLLM_PACKED(rllm_softcap_rows)

@@ -583,7 +583,7 @@ def latent_rope_store(q, kv, kv_norm_w, cs_table, cs_mult, slots, q_att, cache, 
     """Attention through latents, the step between the projections and the attention kernel: kv
     [n, rank + r] (float32, any row stride) -> cache row [normed latent | rotated shared key part];
     q [n, H * (dq + r)] -> the rotated part of every head into q_att[:, h, rank:rank + r].  `pairs`: entry 2i
-    turns with 2i + 1 (else i with i + r/2).  r 0: no rotated parts, no cs_table.  See headwise.cu."""
+    turns with 2i + 1 (else i with i + r/2).  See headwise.cu."""
     _need_cuda(q, kv, kv_norm_w, cs_table, slots, q_att, cache)
     _need_contig(q_att=q_att, cache=cache, slots=slots)
     _rows2d(q, "q"), _rows2d(kv, "kv")
@@ -592,7 +592,7 @@ def latent_rope_store(q, kv, kv_norm_w, cs_table, cs_mult, slots, q_att, cache, 
     assert q_att.shape == (n, H * (rank + r)) and cache.shape[1:] == (1, block_size, rank + r)
     assert cache.dtype == q_att.dtype and slots.dtype == torch.int32 and slots.numel() == n
     assert kv_norm_w.dtype == torch.float32 and kv_norm_w.numel() == rank and kv_norm_w.is_contiguous()
-    assert r == 0 or (cs_table.dtype == torch.float32 and cs_table.shape == (n, r // 2, 2) and cs_table.is_contiguous())
+    assert cs_table.dtype == torch.float32 and cs_table.shape == (n, r // 2, 2) and cs_table.is_contiguous()
     _check(core().rllm_latent_rope_store(
         _ptr(q), c_int(_code(q)), c_longlong(q.stride(0)), _ptr(kv), c_longlong(kv.stride(0)), _ptr(kv_norm_w),
         _ptr(cs_table), c_float(cs_mult), _ptr(slots), _ptr(q_att), _ptr(cache), c_int(_code(q_att)), c_int(n),
@@ -600,6 +600,25 @@ def latent_rope_store(q, kv, kv_norm_w, cs_table, cs_mult, slots, q_att, cache, 
         c_longlong(cache.shape[0] * block_size), _ptr(error_word(q.device)), c_int(1 if pairs else 0), _stream()),
         "latent_rope_store")
     return q_att
+
+
+def latent_norm_store(low, q_norm_w, kv_norm_w, slots, cq, cache, q_rank, rank, block_size, eps, write_kv=True):
+    """Attention through latents without rotated parts, the step behind the down-projection: low [n, q_rank + rank] (float32) ->
+    cq [n, q_rank] the normed query latent (q_rank 0: none), and the cache rows: the normed latent, zeros behind it up to the
+    row's length.  See headwise.cu."""
+    _need_cuda(low, q_norm_w, kv_norm_w, slots, cq, cache)
+    _need_contig(cq=cq, cache=cache, slots=slots)
+    _rows2d(low, "low")
+    n, W = low.shape[0], cache.shape[-1]
+    assert low.dtype == torch.float32 and low.shape[1] == q_rank + rank and cache.shape[1:3] == (1, block_size) and W >= rank
+    assert slots.dtype == torch.int32 and slots.numel() == n
+    assert kv_norm_w.dtype == torch.float32 and kv_norm_w.numel() == rank and kv_norm_w.is_contiguous()
+    if q_rank:
+        assert q_norm_w.dtype == torch.float32 and q_norm_w.numel() == q_rank and cq.shape == (n, q_rank) and cq.dtype == cache.dtype
+    _check(core().rllm_latent_norm_store(
+        _ptr(low), c_longlong(low.stride(0)), _ptr(q_norm_w), _ptr(kv_norm_w), _ptr(slots), _ptr(cq), _ptr(cache),
+        c_int(_code(cache)), c_int(n), c_int(q_rank), c_int(rank), c_int(W), c_float(eps), c_int(1 if write_kv else 0),
+        c_longlong(cache.shape[0] * block_size), _ptr(error_word(low.device)), _stream()), "latent_norm_store")
 
 
 GLU_GELU_TANH = (0.0, 0.0, 0.0)     # the `glu` triple (limit, alpha, shift) of act = tanh-form gelu: alpha 0 selects it

@@ -23,7 +23,9 @@ the window has passed.  The rotation's pair layout is the position part's.
 
 Parameters: hidden_size, num_heads, head_dim, rot_dim, v_head_dim, kv_rank, q_rank, eps, scale,
 softcap, window.  Tensors <prefix>dq, dq.norm, uq (or q), dkv, dkv.norm, uk, uv, o.  Load-time transforms: dq and
-dkv are stacked into one product on h; uk is kept per head and transposed ([H, kv_rank, dq]).
+dkv are stacked into one product on h; uk is kept per head and transposed ([H, kv_rank, dq]).  Without a rotated part,
+bfloat16 cache rows get zeros behind the latent up to a multiple of 64 entries (as do uk and uv), the sizes that the
+tensor-core decode kernel takes.
 Norms, angles, scores and softmax are float32 in every mode.
 """
 from __future__ import annotations
@@ -50,12 +52,15 @@ class LatentAttention(Mixer):
         self.window = int(p.get("window", 0) or 0)
         if self.r < 0 or self.r % 2:
             raise PartError(f"latent_attention: rot_dim {self.r} must be even (0: no rotated part)")
+        self.rank_s = self.rank          # entries of a latent as stored
+        if self.r == 0 and not runtime.is_f32:
+            self.rank_s = -(-self.rank // 64) * 64
         if self.rank > 512 or self.rank + self.r > 2048:
             raise PartError("latent_attention: kv_rank up to 512, kv_rank + rot_dim up to 2048")
         self.w_down = self.w_uq = self.w_qc = self.w_uv = self.w_o = self.q_norm_w = self.kv_norm_w = None
 
     def cache_need(self):
-        return PagedKVNeed(1, self.rank + self.r, window=self.window, values_in_keys=self.rank)
+        return PagedKVNeed(1, self.rank_s + self.r, window=self.window, values_in_keys=self.rank_s)
 
     def expected_tensors(self):
         d, p, H = self.hidden_size, self.prefix, self.H
@@ -77,18 +82,24 @@ class LatentAttention(Mixer):
             self.w_uq = self._to_device(tensors[p + "q"])
         self.kv_norm_w = self._to_device(tensors[p + "dkv.norm"], torch.float32)
         # [H, dq, rank] -> [H, rank, dq]: the product that takes a head's plain query into latent space
-        self.w_qc = self._to_device(tensors[p + "uk"].to(dt).view(self.H, self.dq, self.rank).transpose(1, 2))
-        self.w_uv = self._to_device(tensors[p + "uv"].to(dt).view(self.H, self.dv, self.rank))
+        def wide(t):                     # [H, rows, rank] -> [H, rows, rank_s]
+            return torch.nn.functional.pad(t, (0, self.rank_s - self.rank)) if self.rank_s > self.rank else t
+        self.w_qc = self._to_device(wide(tensors[p + "uk"].to(dt).view(self.H, self.dq, self.rank)).transpose(1, 2))
+        self.w_uv = self._to_device(wide(tensors[p + "uv"].to(dt).view(self.H, self.dv, self.rank)))
         self.w_o = self._to_device(tensors[p + "o"])
 
     def forward(self, h, ctx, cache, position=None, residual=None):
         n, dt, dev = h.shape[0], self.runtime.dtype, h.device
-        H, dq, r, rank = self.H, self.dq, self.r, self.rank
+        H, dq, r, rank = self.H, self.dq, self.r, self.rank_s
         if (position.dims if position is not None else 0) != r:
             raise PartError("latent_attention: needs a rotary position part over rot_dim entries")
         low = ops.linear(h, self.w_down, out_dtype=torch.float32)              # [query latent | c | kr]
-        if self.q_rank:
-            cq = torch.empty((n, self.q_rank), dtype=dt, device=dev)
+        cq = torch.empty((n, self.q_rank), dtype=dt, device=dev) if self.q_rank else None
+        if r == 0:
+            ops.latent_norm_store(low, self.q_norm_w, self.kv_norm_w, cache.slots, cq, cache.k, self.q_rank, self.rank,
+                                  cache.block_size, self.eps, write_kv=cache.write)
+            q = ops.linear(cq if self.q_rank else h, self.w_uq, out_dtype=dt)
+        elif self.q_rank:
             ops.norm_rows(low[:, :self.q_rank], self.q_norm_w, self.eps, low=cq)
             q = ops.linear(cq, self.w_uq, out_dtype=dt)                         # [n, H * (dq + r)]
         else:
@@ -96,9 +107,10 @@ class LatentAttention(Mixer):
         W = rank + r
         q_att = torch.empty((n, H * W), dtype=dt, device=dev)
         ops.head_linear(q.view(n, H, dq + r)[:, :, :dq], self.w_qc, q_att.view(n, H, W)[:, :, :rank])
-        ops.latent_rope_store(q, low[:, self.q_rank:], self.kv_norm_w, position.angles(ctx) if r else None,
-                              position.mult if r else 1.0, cache.slots, q_att, cache.k, H, dq, r, rank, cache.block_size, self.eps,
-                              write_kv=cache.write, pairs=getattr(position, "layout", "half") == "pairs")
+        if r:
+            ops.latent_rope_store(q, low[:, self.q_rank:], self.kv_norm_w, position.angles(ctx), position.mult,
+                                  cache.slots, q_att, cache.k, H, dq, r, rank, cache.block_size, self.eps,
+                                  write_kv=cache.write, pairs=getattr(position, "layout", "half") == "pairs")
         mixed = torch.empty((n, H * rank), dtype=dt, device=dev)
         ops.shared_kv_attention(q_att, cache.k, mixed, ctx, cache.block_table, H, W, rank, cache.block_size,
                                 self.scale, softcap=self.softcap, window=self.window)
