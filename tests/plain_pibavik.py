@@ -161,9 +161,10 @@ def choose(s, top):
     return order[:top], float(s[order[top - 1]] - s[order[top]]) if top < len(order) else math.inf
 
 
-def experts(h, w, pre, mlp, given=None, slack=0.0, margins=None):
+def experts(h, w, pre, mlp, given=None, slack=0.0, margins=None, chosen=None):
     """`given` {token index: experts}: somebody else's choice is taken over for a token when moving every
-    score by at most `slack` makes it this router's own.  `margins` (a list) takes the distances per token."""
+    score by at most `slack` makes it this router's own.  `margins` (a list) takes the distances per token, `chosen`
+    (a dictionary) the experts."""
     r = mlp["router"]
     s = torch.sigmoid(h @ w[pre + "router"].T)
     out = torch.zeros_like(h)
@@ -177,6 +178,8 @@ def experts(h, w, pre, mlp, given=None, slack=0.0, margins=None):
             moved[cand] += 2 * slack
             if sorted(choose(moved, r["top"])[0]) == sorted(cand):
                 idx = cand
+        if chosen is not None:
+            chosen[t] = list(idx)
         for e in idx:
             out[t] += expert(s[t, e] * h[t:t + 1], w, f"{pre}e{e}.")[0]
     if margins is not None:
@@ -200,26 +203,26 @@ def mixer(h, w, i, spec, eps, kv):
     return side_by_side(h, w, pre, mx, eps)
 
 
-def layer(x, w, i, spec, cfg, kv, given=None, slack=0.0, margins=None, coarse=None):
+def layer(x, w, i, spec, cfg, kv, given=None, slack=0.0, margins=None, coarse=None, chosen=None):
     """`coarse`, if given, is applied to what every sublayer reads and returns (operands of fewer bits)."""
     eps = cfg["norm"]["eps"]
     see = coarse or (lambda t: t)
     x = x + see(mixer(see(rms(x, eps) * w[f"l{i}.norm1"]), w, i, spec, eps, kv))
     if spec.get("mlp"):
         x = x + see(experts(see(rms(x, eps) * w[f"l{i}.norm2"]), w, f"l{i}.mlp.", spec["mlp"], (given or {}).get(i), slack,
-                            margins))
+                            margins, chosen.setdefault(i, {}) if chosen is not None else None))
     return x
 
 
-def forward(cfg, weights, tokens, streams=None, margins=None, given=None, slack=0.0, coarse=None):
+def forward(cfg, weights, tokens, streams=None, margins=None, given=None, slack=0.0, coarse=None, chosen=None):
     """Logits [n, vocab] (float64) of one sequence from its start.  `weights`: name -> tensor of any float
     type; `streams`, if a list, takes the stream after every layer; the rest: see `experts` and `layer`
-    (`given` is {layer: {token index: experts}})."""
+    (`given` and `chosen` are {layer: {token index: experts}})."""
     w = {k: v.to(F64) for k, v in weights.items()}
     x = w["embed"][torch.tensor(list(tokens), dtype=torch.long)] * cfg["embedding"]["scale"]
     kv = {}
     for i, spec in enumerate(cfg["layers"]):
-        x = layer(x, w, i, spec, cfg, kv, given, slack, margins, coarse)
+        x = layer(x, w, i, spec, cfg, kv, given, slack, margins, coarse, chosen)
         if streams is not None:
             streams.append(x.clone())
     x = rms(x, cfg["norm"]["eps"]) * w["final.norm"]
