@@ -42,6 +42,7 @@ LIBRARIES = {
     "attn_latent": (["attention_latent.cu"], []),
     "tc": (["gemm_tc.cu"], []),
     "tc2": (["gemm_tc2.cu"], []),
+    "group": (["gemm_group.cu"], []),
     "stream": (["gemv_stream.cu"], []),
     "attn_tc": (["attention_tc.cu"], []),
     "host": (["host_runtime.cpp"], []),

@@ -500,33 +500,38 @@ moe_expert_gate_up_kernel(const bf16* h, const bf16* __restrict__ w_gu, const in
 
 #define MOE_DOWN_COLS 64     // columns per block of the products with one matrix (4 warps, 16 columns a warp)
 
-// act[pair, f] = f(weight[pair] * (Wu[e][f, :] . h[t])) for the pairs of the block's expert; a warp's 16 rows are 16 columns
+// act[pair, f] = f(weight[pair] * (Wu[e][f, :] . h[t])) for the pairs of the block's expert; 16 columns a block, whose four warps
+// take a quarter of k each (many short blocks: an expert's matrix streams through more of them at a time), added in warp order
+#define MOE_UP_COLS 16
 __global__ void __launch_bounds__(128)
 moe_expert_up_kernel(const bf16* h, const bf16* __restrict__ w_up, const int* idx, const float* weight, bf16* act, int n_pairs,
                      int top_k, int d, int F, int act_kind) {
     __shared__ int s_list[MOE_LIST];
     __shared__ int s_n;
+    __shared__ float s_part[4][MOE_UP_COLS * MOE_MT];
     pdl_wait();
     pdl_launch_dependents();
     const int e = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, c = lane & 3;
     const int cnt = list_expert_pairs(idx, n_pairs, e, s_list, &s_n);
     if (cnt == 0) return;
-    const int f_lo = blockIdx.y * MOE_DOWN_COLS + warp * 16 + g, f_hi = f_lo + 8;
-    const bf16* lo = w_up + ((size_t)e * F + min(f_lo, F - 1)) * d;
-    const bf16* hi = w_up + ((size_t)e * F + min(f_hi, F - 1)) * d;
+    const int f0 = blockIdx.y * MOE_UP_COLS;
+    const int share = ((d + 3) / 4 + 127) / 128 * 128, k0 = min(d, warp * share), k1 = min(d, k0 + share);
+    const bf16* lo = w_up + ((size_t)e * F + min(f0 + g, F - 1)) * d + k0;
+    const bf16* hi = w_up + ((size_t)e * F + min(f0 + g + 8, F - 1)) * d + k0;
     for (int c0 = 0; c0 < cnt; c0 += MOE_MT) {
         const int mine = s_list[min(c0 + g, cnt - 1)];
         float acc[4];
-        rows16_times_tokens8(lo, hi, h + (size_t)(mine / top_k) * d, d, c, acc);
+        rows16_times_tokens8(lo, hi, h + (size_t)(mine / top_k) * d + k0, k1 - k0, c, acc);
 #pragma unroll
-        for (int q = 0; q < 2; ++q) {
-            const int at = c0 + 2 * c + q;
-            if (at >= cnt) continue;
+        for (int q = 0; q < 4; ++q) s_part[warp][(2 * c + (q & 1)) * MOE_UP_COLS + g + (q >> 1) * 8] = acc[q];
+        __syncthreads();
+        const int tok = threadIdx.x / MOE_UP_COLS, col = threadIdx.x % MOE_UP_COLS, at = c0 + tok;      // 128 threads: 8 tokens x 16 columns
+        if (at < cnt && f0 + col < F) {
             const size_t pair = s_list[at];
-            const float wt = weight ? weight[pair] : 1.f;
-            if (f_lo < F) act[pair * F + f_lo] = from_f<bf16>(act_apply(wt * acc[q], act_kind));
-            if (f_hi < F) act[pair * F + f_hi] = from_f<bf16>(act_apply(wt * acc[2 + q], act_kind));
+            const float v = s_part[0][threadIdx.x] + s_part[1][threadIdx.x] + s_part[2][threadIdx.x] + s_part[3][threadIdx.x];
+            act[pair * F + f0 + col] = from_f<bf16>(act_apply((weight ? weight[pair] : 1.f) * v, act_kind));
         }
+        __syncthreads();
     }
 }
 
@@ -576,7 +581,7 @@ RLLM_API int rllm_moe_expert_up(const void* h, const void* w_up, const int* idx,
     if (n <= 0) return 0;
     if (d <= 0 || F <= 0 || top_k <= 0 || E <= 0 || !expert_kernels_fit(n, d) || ((uintptr_t)h & 15) || ((uintptr_t)w_up & 15))
         return (int)cudaErrorInvalidValue;
-    return rllm_launch_after(moe_expert_up_kernel, dim3(E, (F + MOE_DOWN_COLS - 1) / MOE_DOWN_COLS), dim3(128), 0, stream,
+    return rllm_launch_after(moe_expert_up_kernel, dim3(E, (F + MOE_UP_COLS - 1) / MOE_UP_COLS), dim3(128), 0, stream,
                              (const bf16*)h, (const bf16*)w_up, idx, weight, (bf16*)act, n * top_k, top_k, d, F, act_kind);
 }
 

@@ -822,20 +822,20 @@ TIME_SEGMENTS = os.environ.get("RLLM_B200_NO_TIME_SEGMENTS", "0") in ("", "0")
 
 class TimeSegments:
     """The step's requests cut along time for the recurrent kernels (recurrent.cu, TimeSegments): a
-    request that brings fewer than SEGMENT_FROM tokens is one item, a longer one several of
-    SEGMENT_TOKENS tokens (the last takes the remainder).  Built once per step on the host from the
+    request that brings fewer than `shortest` tokens is one item, a longer one several of
+    `length` tokens (the last takes the remainder).  Built once per step on the host from the
     step's shape and shared by all layers."""
 
-    def __init__(self, ctx, device):
+    def __init__(self, ctx, device, length=SEGMENT_TOKENS, shortest=SEGMENT_FROM):
         t0, t1, req, flags, item0, items = [], [], [], [], [], []
         base = 0
         for r, q in enumerate(ctx.q_lens):
-            n = q // SEGMENT_TOKENS if q >= SEGMENT_FROM else 1
+            n = q // length if q >= shortest else 1
             item0.append(len(t0))
             items.append(n)
             for s in range(n):
-                t0.append(base + s * SEGMENT_TOKENS)
-                t1.append(base + (s + 1) * SEGMENT_TOKENS if s + 1 < n else base + q)
+                t0.append(base + s * length)
+                t1.append(base + (s + 1) * length if s + 1 < n else base + q)
                 req.append(r)
                 flags.append((1 if s == 0 else 0) | (2 if s + 1 == n else 0))
             base += q
@@ -846,13 +846,14 @@ class TimeSegments:
         self.item0, self.items = flat[4 * n:4 * n + R], flat[4 * n + R:4 * n + 2 * R]
 
 
-def time_segments(ctx, device):
+def time_segments(ctx, device, length=SEGMENT_TOKENS, shortest=SEGMENT_FROM):
     """The step's TimeSegments, or None when no request brings a portion long enough to cut."""
-    if not TIME_SEGMENTS or ctx.max_q_len < SEGMENT_FROM:
+    if not TIME_SEGMENTS or ctx.max_q_len < shortest:
         return None
-    plan = ctx.plans.get("time_segments")
+    key = ("time_segments", length, shortest)
+    plan = ctx.plans.get(key)
     if plan is None:
-        plan = ctx.plans["time_segments"] = TimeSegments(ctx, device)
+        plan = ctx.plans[key] = TimeSegments(ctx, device, length, shortest)
     return plan
 
 
@@ -1060,6 +1061,13 @@ def ssd_state_floats(H: int, P: int, N: int, G: int, taps: int) -> int:
     return (H * P * N + (taps - 1 + SSD_STEP_TOKENS) * (H * P + 2 * G * N) + 3) // 4 * 4
 
 
+def ssd_segment_tokens(H: int, P: int) -> int:
+    """Length of a segment when a long portion is cut along time: a function of the layer's sizes alone, so that a portion of
+    2,048 tokens makes about two blocks per SM (few heads: short segments)."""
+    blocks = H * -(-P // 64)
+    return min(1024, max(128, 8 * blocks // 64 * 64))
+
+
 def ssd(rows, conv, conv_b, dt_bias, A, D, norm_w, eps, norm_groups, state, ctx, slots, out, H, G, P, N):
     """The state-space recurrence with one decay per head behind its convolution, gated and normed; see ssd.cu.  rows: float32
     [n, ...] with z [H*P], the convolution's channels x [H*P], B, C [G*N] each, and dt [H] side by side; conv float32 [taps,
@@ -1078,23 +1086,30 @@ def ssd(rows, conv, conv_b, dt_bias, A, D, norm_w, eps, norm_groups, state, ctx,
         raise KernelError(f"ssd: at most 256 state entries per column, got {N}")
     st = _state2d(state)
     assert ssd_state_floats(H, P, N, G, taps) <= st.shape[1]
-    mode, xbc, dts, ldx = 0, None, None, 0
+    mode, xbc, dts, ldx, sg, carry, decay = 0, None, None, 0, None, None, None
     if ctx.max_q_len > SSD_STEP_TOKENS:
         mode = 2 if out.dtype == torch.bfloat16 else 1
         ldx = H * (-(-P // 8) * 8) + 2 * G * (-(-N // 8) * 8)
         make = torch.empty if P % 8 == 0 and N % 8 == 0 else torch.zeros       # padding entries of a head or group read as zero
         xbc = make((n, ldx), dtype=out.dtype, device=out.device)
         dts = torch.empty((2, H, n), dtype=torch.float32, device=out.device)
+        length = ssd_segment_tokens(H, P)
+        sg = time_segments(ctx, out.device, length, 2 * length) if mode == 2 else None
+        if sg is not None:
+            carry = torch.empty((sg.n_items, H, P, N), dtype=torch.float32, device=out.device)
+            decay = torch.empty((sg.n_items, H), dtype=torch.float32, device=out.device)
     _check(_lib("ssd").rllm_ssd(
         _ptr(rows), c_longlong(rows.stride(0)), c_int(0), c_int(inner), c_int(inner + C), _ptr(conv), _ptr(conv_b), _ptr(dt_bias),
         _ptr(A), _ptr(D), _ptr(st), c_longlong(st.stride(0)), _ptr(ctx.positions), _ptr(ctx.seq_ids), _ptr(ctx.cu_q), _ptr(slots),
         c_int(H), c_int(G), c_int(P), c_int(N), c_int(taps), c_int(n), c_int(ctx.n_requests), c_int(mode), _ptr(xbc),
-        c_longlong(ldx), _ptr(dts), _ptr(out), c_int(_code(out)), c_longlong(out.stride(0)), _stream()), "ssd")
+        c_longlong(ldx), _ptr(dts), _ptr(out), c_int(_code(out)), c_longlong(out.stride(0)), _ptr(sg.t0 if sg else None),
+        _ptr(sg.t1 if sg else None), _ptr(sg.req if sg else None), _ptr(sg.flags if sg else None), _ptr(sg.item0 if sg else None),
+        _ptr(sg.items if sg else None), c_int(sg.n_items if sg else 0), _ptr(carry), _ptr(decay), _stream()), "ssd")
     _check(_lib("ssd").rllm_ssd_norm(_ptr(out), c_int(_code(out)), c_longlong(out.stride(0)), _ptr(norm_w), c_int(n),
                                      c_int(norm_groups), c_int(inner // norm_groups), c_float(eps), _stream()), "ssd_norm")
     if mode:
         global _launches
-        _launches += 1                         # the convolution's kernel
+        _launches += 3 if sg is not None else 1      # the convolution's kernel, the local pass and the carry
     return out
 
 
@@ -1217,6 +1232,33 @@ def moe_gather_rows(h, place, rows, top_k, weight=None, weight_out=None):
                                             c_int(top_k), c_int(h.shape[1]), _ptr(weight), _ptr(weight_out), _stream()),
            "moe_gather_rows")
     return rows
+
+
+def gemm_group_ok(a, w) -> bool:
+    """Whether `gemm_group` takes rows `a` [rows, K] and matrices `w` [E, N, K] or [N, K] (bfloat16, contiguous, K a multiple of 8)."""
+    return (a.dtype == w.dtype == torch.bfloat16 and a.shape[-1] % 8 == 0 and a.is_contiguous() and w.is_contiguous()
+            and a.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0)
+
+
+def gemm_group(a, w, out, offsets=None, row_scale=None, activation=None):
+    """out[r] = f(row_scale[r] * (w[e] . a[r])) for the rows of every expert e, which lie in expert order (offsets int32 [E + 1] on
+    the device); w [E, N, K], or [N, K] without offsets: one matrix for all rows.  row_scale float32 [rows] or None, f by name
+    (ACT); out float32 or bfloat16 [rows, N].  One launch on the tcgen05 tensor cores, whatever the experts' counts; see gemm_group.cu."""
+    _need_cuda(a, w, out, offsets, row_scale)
+    rows, K = a.shape
+    E, N = (w.shape[0], w.shape[1]) if offsets is not None else (1, w.shape[0])
+    if not gemm_group_ok(a, w):
+        raise KernelError("gemm_group takes contiguous bfloat16 rows and matrices whose rows are a multiple of 8 long")
+    assert w.shape[-1] == K and w.dim() == (3 if offsets is not None else 2) and out.shape == (rows, N) and out.stride(1) == 1
+    assert offsets is None or (offsets.dtype == torch.int32 and offsets.numel() == E + 1 and offsets.is_contiguous())
+    assert row_scale is None or (row_scale.dtype == torch.float32 and row_scale.numel() == rows and row_scale.is_contiguous())
+    st = _lib("group").rllm_gemm_group(_ptr(a), _ptr(w), _ptr(out), c_int(_code(out)), c_longlong(out.stride(0)), _ptr(offsets), c_int(E),
+                                       c_int(rows), c_int(N), c_int(K), _ptr(row_scale), c_int(ACT[activation]),
+                                       _ptr(error_word(a.device)), _stream())
+    if st >= 30000:
+        raise KernelError(f"gemm_group: tensor map encoding failed (CUresult {st - 30000})")
+    _check(st, "gemm_group")
+    return out
 
 
 def moe_combine(y, place, weight, out, shared=None, gate=None, top_k=None):
@@ -1426,7 +1468,8 @@ def check_device_errors(device="cuda:0") -> None:
                           f"2 a stage was never released, 3 the accumulator never completed)")
 
 
-_WAIT_LIBRARIES = {"tc": "rllm_tc", "tc2": "rllm_tc2", "stream": "rllm_stream", "attn_tc": "rllm_attn_tc"}
+_WAIT_LIBRARIES = {"tc": "rllm_tc", "tc2": "rllm_tc2", "stream": "rllm_stream", "attn_tc": "rllm_attn_tc",
+                   "group": "rllm_gemm_group"}
 
 
 def set_wait_cycles(cycles: int = 0, libraries=None) -> None:

@@ -21,7 +21,9 @@
 //               the kernel below does not take.
 //   ssd_chunk   bfloat16 portions on the tensor cores, in chunks of 64 tokens counted from the portion's start: a block
 //               per (head, 16 to 64 rows of S, request) walks the request's chunks with S^T in the accumulators of
-//               mma.sync.  With L_i = log(a_1 .. a_i) of a chunk:
+//               mma.sync (two warps, the halves of N, per 16 rows).  Long portions are also cut along time: pass 1 works
+//               out what every segment's tokens leave from an empty state, ssd_carry the state that every segment starts
+//               from, pass 2 the outputs, all segments side by side.  With L_i = log(a_1 .. a_i) of a chunk:
 //                   y_i = e^(L_i) S0 C_i + sum_(j<=i) (C_i . B_j) e^(L_i - L_j) d_j x_j
 //                   S   = e^(L_64) S0 + sum_j e^(L_64 - L_j) d_j x_j B_j^T
 //               x, B and C are bfloat16 as stored; every other operand (S0, the weighted scores, the weighted x) goes into
@@ -137,18 +139,17 @@ ssd_conv_kernel(const SsdArgs p, TA* xbc, long long ldx, float* dts, int n) {
 #pragma unroll
         for (int j = 0; j < TAPS; ++j) w[j] = ssd_load<VEC>(p.conv + (size_t)j * C + c);
         int req = -1;
-        for (int t = t0; t < t1; ++t) {
-            const int r = p.seq_ids[t];
-            if (r != req) {                                   // a request's first token here: its window from the row or the ring
-                const int i = t - p.cu_q[r], pos = p.positions[t];
-                const float* ring = p.state + (size_t)p.slots[r] * p.slot_stride + p.ring_base;
+        auto open_window = [&](int t, int r) {                // a request's first token here: its window from the row or the ring
+            const int i = t - p.cu_q[r], pos = p.positions[t];
+            const float* ring = p.state + (size_t)p.slots[r] * p.slot_stride + p.ring_base;
 #pragma unroll
-                for (int j = 0; j < TAPS - 1; ++j) win[j + 1] = input(ring, t, i, pos, TAPS - 1 - j);
-                req = r;
-            }
+            for (int j = 0; j < TAPS - 1; ++j) win[j + 1] = input(ring, t, i, pos, TAPS - 1 - j);
+            req = r;
+        };
+        auto token = [&](int t, const SsdVec<VEC>& x) {
 #pragma unroll
             for (int j = 0; j < TAPS - 1; ++j) win[j] = win[j + 1];
-            win[TAPS - 1] = ssd_load<VEC>(src + (size_t)t * p.ld);
+            win[TAPS - 1] = x;
             SsdVec<VEC> acc = bias;
 #pragma unroll
             for (int j = 0; j < TAPS; ++j)
@@ -157,6 +158,22 @@ ssd_conv_kernel(const SsdArgs p, TA* xbc, long long ldx, float* dts, int n) {
 #pragma unroll
             for (int q = 0; q < VEC; ++q) acc.v[q] = silu_f(acc.v[q]);
             ssd_put<VEC>(xbc + (size_t)t * ldx + col, acc);
+        };
+        if (t1 - t0 == SSD_CONV_TOK && p.seq_ids[t0] == p.seq_ids[t1 - 1]) {      // one request: the inputs of eight tokens in flight
+            open_window(t0, p.seq_ids[t0]);
+            for (int t = t0; t < t1; t += 8) {
+                SsdVec<VEC> x[8];
+#pragma unroll
+                for (int u = 0; u < 8; ++u) x[u] = ssd_load<VEC>(src + (size_t)(t + u) * p.ld);
+#pragma unroll
+                for (int u = 0; u < 8; ++u) token(t + u, x[u]);
+            }
+            return;
+        }
+        for (int t = t0; t < t1; ++t) {
+            const int r = p.seq_ids[t];
+            if (r != req) open_window(t, r);
+            token(t, ssd_load<VEC>(src + (size_t)t * p.ld));
         }
     } else {
         for (int t = t0; t < t1; ++t) {
@@ -179,7 +196,7 @@ ssd_conv_kernel(const SsdArgs p, TA* xbc, long long ldx, float* dts, int n) {
 // LN lanes share a row of S (KV runs of VEC entries a lane); RU rows a lane group at a time.  FUSED: the step has at
 // most SSD_STEP tokens a request and the kernel does the convolution and the step sizes itself; else xbc and dts.
 template <typename TA, int VEC, int KV, bool FUSED>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(256, 3)
 ssd_step_kernel(const SsdArgs p, const TA* xbc, long long ldx, const float* dts, int n, TA* out, long long ldo, int LN) {
     constexpr int RU = 8 / KV;
     extern __shared__ __align__(16) float sm_ssd[];
@@ -253,8 +270,10 @@ ssd_step_kernel(const SsdArgs p, const TA* xbc, long long ldx, const float* dts,
             s_d[SSD_STEP + tid] = expf(la);
         }
         __syncthreads();
-        for (int p0 = grp; p0 < p.P; p0 += groups * RU) {
-            if (p0 != grp) load(p0);
+        // every lane goes through every round, also one whose rows lie beyond P: the sums below are warp-wide
+        for (int base = 0; base < p.P; base += groups * RU) {
+            const int p0 = base + grp;
+            if (base) load(p0);
             for (int i = 0; i < cnt; ++i) {
                 const float d = s_d[i], a = s_d[SSD_STEP + i];
                 SsdVec<VEC> b[KV], cc[KV];
@@ -351,55 +370,72 @@ __device__ __forceinline__ void ssd_split(float x, float y, uint32_t& hi, uint32
 }
 __device__ __forceinline__ float2 ssd_pair(uint32_t u) { return __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u)); }
 
-template <int NK> struct SsdTile {                   // N padded to 16 * NK
-    static constexpr int NS = NK * 16 + 8;           // row stride of B and C (a shift of 16 bytes a row: ldmatrix without conflicts)
-    static constexpr int MS = SSD_CHUNK + 8;         // of the weighted scores
-    __host__ __device__ static constexpr int PS(int W) { return 16 * W + 8; }
-    __host__ __device__ static constexpr int YS(int W) { return 16 * W + 4; }
-    __host__ __device__ static constexpr size_t stage(int W) { return (size_t)SSD_CHUNK * (2 * NS + PS(W)) * sizeof(bf16); }
-    __host__ __device__ static constexpr size_t bytes(int W) {
-        return 2 * stage(W) + 2 * SSD_CHUNK * MS * sizeof(bf16) + (size_t)SSD_CHUNK * YS(W) * sizeof(float) +
-               2 * 2 * SSD_CHUNK * sizeof(float);
-    }
+// Segments of the step's requests along time (all null: every request is one item).
+struct SsdSegments {
+    const int* t0;        // [items] first flat token
+    const int* t1;        // [items] one past the last
+    const int* req;       // [items] the request's row in the step
+    const int* flags;     // [items] bit 0: first segment of its request, bit 1: last
+    const int* item0;     // [requests] a request's first item
+    const int* items;     // [requests] how many it has
+    float* carry;         // [items][H][P][N]: what a segment's tokens leave from an empty state, then the state it starts from
+    float* decay;         // [items][H]: the sum of the segment's log decays
 };
 
-template <int NK, int W>
-__global__ void __launch_bounds__(W * 32, NK <= 8 ? 2 : 1)
-ssd_chunk_kernel(const SsdArgs p, const bf16* xbc, long long ldx, const float* dts, int n, bf16* out, long long ldo) {
-    using Tile = SsdTile<NK>;
-    constexpr int Q = SSD_CHUNK, NS = Tile::NS, MS = Tile::MS, PS = Tile::PS(W), YS = Tile::YS(W), NT = W * 32;
+template <int NK, int PW> struct SsdTile {           // N padded to 16 * NK, 16 * PW rows of S^T
+    static constexpr int NT = PW * 64;               // threads: two warps (halves of N) per 16 rows
+    static constexpr int NS = NK * 16 + 8;           // row stride of B and C (a shift of 16 bytes a row: ldmatrix without conflicts)
+    static constexpr int MS = SSD_CHUNK + 8;         // of the weighted scores
+    static constexpr int PS = 16 * PW + 8;           // of x
+    static constexpr int YS = 16 * PW + 4;           // of the outputs (over the weighted scores)
+    static constexpr size_t stage = (size_t)SSD_CHUNK * (2 * NS + PS) * sizeof(bf16);
+    static constexpr size_t m_bytes = 2 * SSD_CHUNK * MS * sizeof(bf16), y_bytes = (size_t)SSD_CHUNK * YS * sizeof(float);
+    static constexpr size_t bytes = 2 * stage + (m_bytes > y_bytes ? m_bytes : y_bytes) + 2 * 2 * SSD_CHUNK * sizeof(float);
+};
+
+// PASS 0: whole requests.  1: what the tokens of a segment leave from an empty state, and their decay; no output.  2: segments
+// from the state they start from, with output.
+template <int NK, int PW, int PASS>
+__global__ void __launch_bounds__(PW * 64, NK <= 8 ? 8 / PW : 4 / PW)
+ssd_chunk_kernel(const SsdArgs p, const bf16* xbc, long long ldx, const float* dts, int n, bf16* out, long long ldo,
+                 const SsdSegments seg) {
+    using Tile = SsdTile<NK, PW>;
+    constexpr int Q = SSD_CHUNK, NS = Tile::NS, MS = Tile::MS, PS = Tile::PS, YS = Tile::YS, NT = Tile::NT, NH = NK / 2, NW = NT / 32;
     extern __shared__ __align__(128) unsigned char sm_raw[];
-    bf16* s_m = reinterpret_cast<bf16*>(sm_raw + 2 * Tile::stage(W));         // [2][Q][MS]: high and low parts
-    float* s_y = reinterpret_cast<float*>(s_m + 2 * Q * MS);                  // [Q][YS]
-    float* s_d = s_y + Q * YS;                                                // [2 stages][2][Q]: step sizes, sums of log decays
+    bf16* s_m = reinterpret_cast<bf16*>(sm_raw + 2 * Tile::stage);            // [2][Q][MS]: high and low parts
+    float* s_y = reinterpret_cast<float*>(s_m);                               // [Q][YS], when the scores have been read
+    float* s_d = reinterpret_cast<float*>(sm_raw + Tile::bytes) - 4 * Q;      // [2 stages][2][Q]: step sizes, sums of log decays
     // (no early launch of what follows while the long-lived blocks are still to be placed)
     pdl_wait();
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g8 = lane >> 2, c2 = (lane & 3) * 2;
-    const int mi = lane >> 3, ri = lane & 7;
-    const int tiles = (p.P + 16 * W - 1) / (16 * W), h = blockIdx.x / tiles, p0 = (blockIdx.x % tiles) * 16 * W, r = blockIdx.y;
+    const int mi = lane >> 3, ri = lane & 7, pw = warp >> 1, half = warp & 1;
+    const int tiles = (p.P + 16 * PW - 1) / (16 * PW), h = blockIdx.x / tiles, p0 = (blockIdx.x % tiles) * 16 * PW;
+    const int item = blockIdx.y, r = PASS == 0 ? item : seg.req[item];
+    const int t0 = PASS == 0 ? p.cu_q[r] : seg.t0[item], len = (PASS == 0 ? p.cu_q[r + 1] : seg.t1[item]) - t0;
+    const bool first = PASS == 0 || (seg.flags[item] & 1), last = PASS == 0 || (seg.flags[item] & 2);
+    if (len <= 0 || (PASS == 1 && last)) return;             // a request's last segment leaves its state in pass 2
     const int grp = h / (p.H / p.G), P8 = ssd_pad8(p.P), N8 = ssd_pad8(p.N);
-    const int t0 = p.cu_q[r], len = p.cu_q[r + 1] - t0;
-    if (len <= 0) return;
     float* slot = p.state + (size_t)p.slots[r] * p.slot_stride;
     float* Sg = slot + (size_t)h * p.P * p.N;
+    float* Sc = PASS == 0 ? nullptr : seg.carry + ((size_t)item * p.H + h) * p.P * p.N;
     float* ring = slot + p.ring_base;
 
     const bf16* x_src = xbc + (size_t)t0 * ldx + (size_t)h * P8 + p0;
     const bf16* b_src = xbc + (size_t)t0 * ldx + (size_t)p.H * P8 + (size_t)grp * N8;
     const bf16* c_src = b_src + (size_t)p.G * N8;
-    const int x_runs = min(P8 - p0, 16 * W) / 8, n_runs = N8 / 8;
+    const int x_runs = min(P8 - p0, 16 * PW) / 8, n_runs = N8 / 8;
     auto fetch = [&](int buf, int c0) {
-        bf16* s_b = reinterpret_cast<bf16*>(sm_raw + buf * Tile::stage(W));
+        bf16* s_b = reinterpret_cast<bf16*>(sm_raw + buf * Tile::stage);
         bf16 *s_c = s_b + Q * NS, *s_x = s_c + Q * NS;
         for (int e = tid; e < Q * 2 * NK; e += NT) {
             const int i = e / (2 * NK), q = e % (2 * NK);
             const bool ok = c0 + i < len && q < n_runs;
             const size_t off = ok ? (size_t)(c0 + i) * ldx + 8 * q : 0;
             ssd_cp16(s_b + i * NS + 8 * q, b_src + off, ok ? 16 : 0);
-            ssd_cp16(s_c + i * NS + 8 * q, c_src + off, ok ? 16 : 0);
+            if (PASS != 1) ssd_cp16(s_c + i * NS + 8 * q, c_src + off, ok ? 16 : 0);
         }
-        for (int e = tid; e < Q * 2 * W; e += NT) {
-            const int i = e / (2 * W), q = e % (2 * W);
+        for (int e = tid; e < Q * 2 * PW; e += NT) {
+            const int i = e / (2 * PW), q = e % (2 * PW);
             const bool ok = c0 + i < len && q < x_runs;
             ssd_cp16(s_x + i * PS + 8 * q, x_src + (ok ? (size_t)(c0 + i) * ldx + 8 * q : 0), ok ? 16 : 0);
         }
@@ -424,107 +460,116 @@ ssd_chunk_kernel(const SsdArgs p, const bf16* xbc, long long ldx, const float* d
         s[Q + i + 1] = run;
     };
     fetch(0, 0);
-    if (warp == W - 1) scan(0, 0);
+    if (warp == NW - 1) scan(0, 0);
 
-    // S^T rows row0 and row0 + 8 of this lane, columns 8 j + c2, + 1
-    const int row0 = p0 + warp * 16 + g8;
-    float S[2 * NK][4];
+    // S^T: rows row0 and row0 + 8 of this lane, columns n0 + 8 j + c2, + 1 (the warp's half of N)
+    const int row0 = p0 + pw * 16 + g8, n0 = half * NH * 16;
+    float S[2 * NH][4];
+    const float* S_from = (PASS == 2 && !(first && last)) ? Sc : Sg;      // (the slot's own state is what the last segment overwrites)
 #pragma unroll
-    for (int j = 0; j < 2 * NK; ++j)
+    for (int j = 0; j < 2 * NH; ++j)
 #pragma unroll
         for (int q = 0; q < 4; ++q) {
-            const int row = row0 + (q >> 1) * 8, c = 8 * j + c2 + (q & 1);
-            S[j][q] = row < p.P && c < p.N ? Sg[(size_t)row * p.N + c] : 0.f;
+            const int row = row0 + (q >> 1) * 8, c = n0 + 8 * j + c2 + (q & 1);
+            S[j][q] = PASS != 1 && row < p.P && c < p.N ? S_from[(size_t)row * p.N + c] : 0.f;
         }
     const float Dh = p.D[h];
+    const bool vec = p.P % 8 == 0 && p.ld % 4 == 0 && p.z_off % 4 == 0 && ldo % 8 == 0 && ((uintptr_t)p.rows & 15) == 0 &&
+                     ((uintptr_t)out & 15) == 0;
+    float total_all = 0.f;
 
     int buf = 0;
     for (int c0 = 0; c0 < len; c0 += Q, buf ^= 1) {
         const int cnt = min(Q, len - c0), it16 = (cnt + 15) / 16;        // runs of 16 tokens that hold something
         asm volatile("cp.async.wait_group 0;\n" ::);
-        __syncthreads();                             // this chunk is there, and everybody is done with the other stage
+        __syncthreads();                             // this chunk is there, and everybody is done with the other stage and the outputs
         if (c0 + Q < len) fetch(buf ^ 1, c0 + Q);
-        const bf16* s_b = reinterpret_cast<const bf16*>(sm_raw + buf * Tile::stage(W));
+        const bf16* s_b = reinterpret_cast<const bf16*>(sm_raw + buf * Tile::stage);
         const bf16 *s_c = s_b + Q * NS, *s_x = s_c + Q * NS;
         const float *s_dt = s_d + buf * 2 * Q, *s_l = s_dt + Q;
+        const float total = s_l[Q - 1], carry = expf(total);
+        float y[8][4];
 
-        // weighted scores: a warp takes runs of 16 tokens i
-        for (int ti = warp; ti < it16; ti += W) {
-            float acc[8][4];
+        if (PASS != 1) {
+            // weighted scores: a warp takes a run of 16 tokens i against 32 tokens j at a time
+            for (int task = warp; task < 8; task += NW) {
+                const int ti = task >> 1, jh = task & 1;
+                if (ti >= it16 || (jh && ti < 2)) continue;
+                float acc[4][4];
 #pragma unroll
-            for (int j = 0; j < 8; ++j) acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f;
+                for (int j = 0; j < 4; ++j) acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f;
 #pragma unroll
-            for (int k = 0; k < NK; ++k) {
-                uint32_t a[4];
-                ssd_ldsm(s_c + (ti * 16 + (mi & 1) * 8 + ri) * NS + k * 16 + (mi >> 1) * 8, a);
+                for (int k = 0; k < NK; ++k) {
+                    uint32_t a[4];
+                    ssd_ldsm(s_c + (ti * 16 + (mi & 1) * 8 + ri) * NS + k * 16 + (mi >> 1) * 8, a);
 #pragma unroll
-                for (int jp = 0; jp < 4; ++jp) {
-                    if (jp <= ti) {
-                        uint32_t b[4];
-                        ssd_ldsm(s_b + (jp * 16 + (mi >> 1) * 8 + ri) * NS + k * 16 + (mi & 1) * 8, b);
-                        ssd_mma(acc[2 * jp], a, b[0], b[1]);
-                        ssd_mma(acc[2 * jp + 1], a, b[2], b[3]);
+                    for (int jq = 0; jq < 2; ++jq) {
+                        const int jp = 2 * jh + jq;
+                        if (jp <= ti) {
+                            uint32_t b[4];
+                            ssd_ldsm(s_b + (jp * 16 + (mi >> 1) * 8 + ri) * NS + k * 16 + (mi & 1) * 8, b);
+                            ssd_mma(acc[2 * jq], a, b[0], b[1]);
+                            ssd_mma(acc[2 * jq + 1], a, b[2], b[3]);
+                        }
+                    }
+                }
+                const int i0 = ti * 16 + g8, i1 = i0 + 8;
+                const float li0 = s_l[i0], li1 = s_l[i1];
+#pragma unroll
+                for (int j = 0; j < 4; ++j) {
+                    const int jc = 32 * jh + 8 * j + c2;
+                    if (2 * jh + (j >> 1) <= ti) {
+                        const float2 lj = *reinterpret_cast<const float2*>(s_l + jc), dj = *reinterpret_cast<const float2*>(s_dt + jc);
+                        const float v00 = jc <= i0 ? acc[j][0] * expf(li0 - lj.x) * dj.x : 0.f;
+                        const float v01 = jc + 1 <= i0 ? acc[j][1] * expf(li0 - lj.y) * dj.y : 0.f;
+                        const float v10 = jc <= i1 ? acc[j][2] * expf(li1 - lj.x) * dj.x : 0.f;
+                        const float v11 = jc + 1 <= i1 ? acc[j][3] * expf(li1 - lj.y) * dj.y : 0.f;
+                        uint32_t hi, lo;
+                        ssd_split(v00, v01, hi, lo);
+                        *reinterpret_cast<uint32_t*>(s_m + i0 * MS + jc) = hi;
+                        *reinterpret_cast<uint32_t*>(s_m + (Q + i0) * MS + jc) = lo;
+                        ssd_split(v10, v11, hi, lo);
+                        *reinterpret_cast<uint32_t*>(s_m + i1 * MS + jc) = hi;
+                        *reinterpret_cast<uint32_t*>(s_m + (Q + i1) * MS + jc) = lo;
                     }
                 }
             }
-            const int i0 = ti * 16 + g8, i1 = i0 + 8;
-            const float li0 = s_l[i0], li1 = s_l[i1];
+            __syncthreads();
+
+            // y^T: what the warp's half of the state before the chunk gives, times e^(L_i), then half of the chunk's own tokens
+#pragma unroll
+            for (int j = 0; j < 8; ++j) y[j][0] = y[j][1] = y[j][2] = y[j][3] = 0.f;
+#pragma unroll
+            for (int k = 0; k < NH; ++k) {
+                uint32_t ah[4], al[4];
+                ssd_split(S[2 * k][0], S[2 * k][1], ah[0], al[0]);
+                ssd_split(S[2 * k][2], S[2 * k][3], ah[1], al[1]);
+                ssd_split(S[2 * k + 1][0], S[2 * k + 1][1], ah[2], al[2]);
+                ssd_split(S[2 * k + 1][2], S[2 * k + 1][3], ah[3], al[3]);
+#pragma unroll
+                for (int ip = 0; ip < 4; ++ip) {
+                    if (ip < it16) {
+                        uint32_t b[4];
+                        ssd_ldsm(s_c + (ip * 16 + (mi >> 1) * 8 + ri) * NS + n0 + k * 16 + (mi & 1) * 8, b);
+                        ssd_mma(y[2 * ip], ah, b[0], b[1]);
+                        ssd_mma(y[2 * ip + 1], ah, b[2], b[3]);
+                        ssd_mma(y[2 * ip], al, b[0], b[1]);
+                        ssd_mma(y[2 * ip + 1], al, b[2], b[3]);
+                    }
+                }
+            }
 #pragma unroll
             for (int j = 0; j < 8; ++j) {
-                if (j <= 2 * ti + 1) {
-                    const int jc = 8 * j + c2;
-                    const float2 lj = *reinterpret_cast<const float2*>(s_l + jc), dj = *reinterpret_cast<const float2*>(s_dt + jc);
-                    const float v00 = jc <= i0 ? acc[j][0] * expf(li0 - lj.x) * dj.x : 0.f;
-                    const float v01 = jc + 1 <= i0 ? acc[j][1] * expf(li0 - lj.y) * dj.y : 0.f;
-                    const float v10 = jc <= i1 ? acc[j][2] * expf(li1 - lj.x) * dj.x : 0.f;
-                    const float v11 = jc + 1 <= i1 ? acc[j][3] * expf(li1 - lj.y) * dj.y : 0.f;
-                    uint32_t hi, lo;
-                    ssd_split(v00, v01, hi, lo);
-                    *reinterpret_cast<uint32_t*>(s_m + i0 * MS + jc) = hi;
-                    *reinterpret_cast<uint32_t*>(s_m + (Q + i0) * MS + jc) = lo;
-                    ssd_split(v10, v11, hi, lo);
-                    *reinterpret_cast<uint32_t*>(s_m + i1 * MS + jc) = hi;
-                    *reinterpret_cast<uint32_t*>(s_m + (Q + i1) * MS + jc) = lo;
-                }
-            }
-        }
-        __syncthreads();
-
-        // y^T: what the state before the chunk gives, times e^(L_i), then the chunk's own tokens
-        float y[8][4];
-#pragma unroll
-        for (int j = 0; j < 8; ++j) y[j][0] = y[j][1] = y[j][2] = y[j][3] = 0.f;
-#pragma unroll
-        for (int k = 0; k < NK; ++k) {
-            uint32_t ah[4], al[4];
-            ssd_split(S[2 * k][0], S[2 * k][1], ah[0], al[0]);
-            ssd_split(S[2 * k][2], S[2 * k][3], ah[1], al[1]);
-            ssd_split(S[2 * k + 1][0], S[2 * k + 1][1], ah[2], al[2]);
-            ssd_split(S[2 * k + 1][2], S[2 * k + 1][3], ah[3], al[3]);
-#pragma unroll
-            for (int ip = 0; ip < 4; ++ip) {
-                if (ip < it16) {
-                    uint32_t b[4];
-                    ssd_ldsm(s_c + (ip * 16 + (mi >> 1) * 8 + ri) * NS + k * 16 + (mi & 1) * 8, b);
-                    ssd_mma(y[2 * ip], ah, b[0], b[1]);
-                    ssd_mma(y[2 * ip + 1], ah, b[2], b[3]);
-                    ssd_mma(y[2 * ip], al, b[0], b[1]);
-                    ssd_mma(y[2 * ip + 1], al, b[2], b[3]);
-                }
+                const float2 l = *reinterpret_cast<const float2*>(s_l + 8 * j + c2);
+                const float e0 = expf(l.x), e1 = expf(l.y);
+                y[j][0] *= e0;
+                y[j][1] *= e1;
+                y[j][2] *= e0;
+                y[j][3] *= e1;
             }
         }
 #pragma unroll
-        for (int j = 0; j < 8; ++j) {
-            const float2 l = *reinterpret_cast<const float2*>(s_l + 8 * j + c2);
-            const float e0 = expf(l.x), e1 = expf(l.y);
-            y[j][0] *= e0;
-            y[j][1] *= e1;
-            y[j][2] *= e0;
-            y[j][3] *= e1;
-        }
-        const float total = s_l[Q - 1], carry = expf(total);
-#pragma unroll
-        for (int j = 0; j < 2 * NK; ++j) {
+        for (int j = 0; j < 2 * NH; ++j) {
             S[j][0] *= carry;
             S[j][1] *= carry;
             S[j][2] *= carry;
@@ -534,18 +579,20 @@ ssd_chunk_kernel(const SsdArgs p, const bf16* xbc, long long ldx, const float* d
         for (int kj = 0; kj < 4; ++kj) {
             if (kj < it16) {
                 uint32_t x[4];
-                ssd_ldsm_t(s_x + (kj * 16 + (mi >> 1) * 8 + ri) * PS + warp * 16 + (mi & 1) * 8, x);
+                ssd_ldsm_t(s_x + (kj * 16 + (mi >> 1) * 8 + ri) * PS + pw * 16 + (mi & 1) * 8, x);
+                if (PASS != 1 && (kj & 1) == half) {
 #pragma unroll
-                for (int ip = 0; ip < 4; ++ip) {
-                    if (ip >= kj && ip < it16) {
-                        uint32_t b[4];
-                        const bf16* at = s_m + (ip * 16 + (mi >> 1) * 8 + ri) * MS + kj * 16 + (mi & 1) * 8;
-                        ssd_ldsm(at, b);
-                        ssd_mma(y[2 * ip], x, b[0], b[1]);
-                        ssd_mma(y[2 * ip + 1], x, b[2], b[3]);
-                        ssd_ldsm(at + Q * MS, b);
-                        ssd_mma(y[2 * ip], x, b[0], b[1]);
-                        ssd_mma(y[2 * ip + 1], x, b[2], b[3]);
+                    for (int ip = 0; ip < 4; ++ip) {
+                        if (ip >= kj && ip < it16) {
+                            uint32_t b[4];
+                            const bf16* at = s_m + (ip * 16 + (mi >> 1) * 8 + ri) * MS + kj * 16 + (mi & 1) * 8;
+                            ssd_ldsm(at, b);
+                            ssd_mma(y[2 * ip], x, b[0], b[1]);
+                            ssd_mma(y[2 * ip + 1], x, b[2], b[3]);
+                            ssd_ldsm(at + Q * MS, b);
+                            ssd_mma(y[2 * ip], x, b[0], b[1]);
+                            ssd_mma(y[2 * ip + 1], x, b[2], b[3]);
+                        }
                     }
                 }
                 // the tokens' part of the new state: x weighted by e^(L_64 - L_j) d_j
@@ -564,9 +611,9 @@ ssd_chunk_kernel(const SsdArgs p, const bf16* xbc, long long ldx, const float* d
                 f = ssd_pair(x[3]);
                 ssd_split(f.x * w2, f.y * w3, xh[3], xl[3]);
 #pragma unroll
-                for (int k = 0; k < NK; ++k) {
+                for (int k = 0; k < NH; ++k) {
                     uint32_t b[4];
-                    ssd_ldsm_t(s_b + (kj * 16 + (mi & 1) * 8 + ri) * NS + k * 16 + (mi >> 1) * 8, b);
+                    ssd_ldsm_t(s_b + (kj * 16 + (mi & 1) * 8 + ri) * NS + n0 + k * 16 + (mi >> 1) * 8, b);
                     ssd_mma(S[2 * k], xh, b[0], b[1]);
                     ssd_mma(S[2 * k + 1], xh, b[2], b[3]);
                     ssd_mma(S[2 * k], xl, b[0], b[1]);
@@ -574,37 +621,104 @@ ssd_chunk_kernel(const SsdArgs p, const bf16* xbc, long long ldx, const float* d
                 }
             }
         }
-        // out: the warp's 16 columns of every token through shared memory
+        total_all += total;
+        if (warp == NW - 1 && c0 + Q < len) scan(buf ^ 1, c0 + Q);
+        if (PASS == 1) continue;
+        // out: the halves added in shared memory (in the order of the halves), then eight columns of a token at a time
+        __syncthreads();                             // the weighted scores have been read
+        if (half == 0) {
 #pragma unroll
-        for (int j = 0; j < 8; ++j)
+            for (int j = 0; j < 8; ++j)
 #pragma unroll
-            for (int q = 0; q < 4; ++q) s_y[(8 * j + c2 + (q & 1)) * YS + warp * 16 + g8 + (q >> 1) * 8] = y[j][q];
-        __syncwarp();
-        for (int e = lane; e < cnt * 2; e += 32) {
-            const int i = e >> 1, c = warp * 16 + (e & 1) * 8, col = p0 + c;
-            const size_t t = t0 + c0 + i;
-            const float* z = p.rows + t * p.ld + p.z_off + (size_t)h * p.P + col;
-            bf16* o = out + t * ldo + (size_t)h * p.P + col;
-#pragma unroll
-            for (int q = 0; q < 8; ++q)
-                if (col + q < p.P)
-                    o[q] = __float2bfloat16_rn((s_y[i * YS + c + q] + Dh * __bfloat162float(s_x[i * PS + c + q])) * silu_f(z[q]));
+                for (int q = 0; q < 4; ++q) s_y[(8 * j + c2 + (q & 1)) * YS + pw * 16 + g8 + (q >> 1) * 8] = y[j][q];
         }
-        if (warp == W - 1 && c0 + Q < len) scan(buf ^ 1, c0 + Q);
+        __syncthreads();
+        if (half == 1) {
+#pragma unroll
+            for (int j = 0; j < 8; ++j)
+#pragma unroll
+                for (int q = 0; q < 4; ++q) s_y[(8 * j + c2 + (q & 1)) * YS + pw * 16 + g8 + (q >> 1) * 8] += y[j][q];
+        }
+        __syncthreads();
+        for (int e = tid; e < cnt * 2 * PW; e += NT) {
+            const int i = e / (2 * PW), c = (e % (2 * PW)) * 8, col = p0 + c;
+            if (col >= p.P) continue;
+            const size_t t = t0 + c0 + i;
+            const float* zp = p.rows + t * p.ld + p.z_off + (size_t)h * p.P + col;
+            bf16* o = out + t * ldo + (size_t)h * p.P + col;
+            const uint4 xu = *reinterpret_cast<const uint4*>(s_x + i * PS + c);
+            const float2 x0 = ssd_pair(xu.x), x1 = ssd_pair(xu.y), x2 = ssd_pair(xu.z), x3 = ssd_pair(xu.w);
+            const float xs[8] = {x0.x, x0.y, x1.x, x1.y, x2.x, x2.y, x3.x, x3.y};
+            float z[8], v[8];
+            if (vec) {
+                const float4 za = *reinterpret_cast<const float4*>(zp), zb = *reinterpret_cast<const float4*>(zp + 4);
+                z[0] = za.x; z[1] = za.y; z[2] = za.z; z[3] = za.w;
+                z[4] = zb.x; z[5] = zb.y; z[6] = zb.z; z[7] = zb.w;
+            } else {
+#pragma unroll
+                for (int q = 0; q < 8; ++q) z[q] = col + q < p.P ? zp[q] : 0.f;
+            }
+            const float4 ya = *reinterpret_cast<const float4*>(s_y + i * YS + c), yb = *reinterpret_cast<const float4*>(s_y + i * YS + c + 4);
+            const float ys[8] = {ya.x, ya.y, ya.z, ya.w, yb.x, yb.y, yb.z, yb.w};
+#pragma unroll
+            for (int q = 0; q < 8; ++q) v[q] = (ys[q] + Dh * xs[q]) * silu_f(z[q]);
+            if (vec) {
+                uint4 u;
+                const __nv_bfloat162 a = __floats2bfloat162_rn(v[0], v[1]), b = __floats2bfloat162_rn(v[2], v[3]);
+                const __nv_bfloat162 cc = __floats2bfloat162_rn(v[4], v[5]), d = __floats2bfloat162_rn(v[6], v[7]);
+                u.x = *reinterpret_cast<const uint32_t*>(&a);
+                u.y = *reinterpret_cast<const uint32_t*>(&b);
+                u.z = *reinterpret_cast<const uint32_t*>(&cc);
+                u.w = *reinterpret_cast<const uint32_t*>(&d);
+                *reinterpret_cast<uint4*>(o) = u;
+            } else {
+#pragma unroll
+                for (int q = 0; q < 8; ++q)
+                    if (col + q < p.P) o[q] = __float2bfloat16_rn(v[q]);
+            }
+        }
     }
     pdl_launch_dependents();
+    if (PASS != 2 || last) {
+        float* S_to = PASS == 1 ? Sc : Sg;
 #pragma unroll
-    for (int j = 0; j < 2 * NK; ++j)
+        for (int j = 0; j < 2 * NH; ++j)
 #pragma unroll
-        for (int q = 0; q < 4; ++q) {
-            const int row = row0 + (q >> 1) * 8, c = 8 * j + c2 + (q & 1);
-            if (row < p.P && c < p.N) Sg[(size_t)row * p.N + c] = S[j][q];
-        }
-    ssd_keep(p, ring, t0, len, h * p.P + p0, min(16 * W, p.P - p0), tid, NT);
+            for (int q = 0; q < 4; ++q) {
+                const int row = row0 + (q >> 1) * 8, c = n0 + 8 * j + c2 + (q & 1);
+                if (row < p.P && c < p.N) S_to[(size_t)row * p.N + c] = S[j][q];
+            }
+    }
+    if (PASS == 1) {
+        if (tid == 0 && p0 == 0) seg.decay[(size_t)item * p.H + h] = total_all;
+        return;
+    }
+    if (!last) return;
+    ssd_keep(p, ring, p.cu_q[r], p.cu_q[r + 1] - p.cu_q[r], h * p.P + p0, min(16 * PW, p.P - p0), tid, NT);
     if (h % (p.H / p.G) == 0 && p0 == 0) {
-        const int inner = p.H * p.P;
-        ssd_keep(p, ring, t0, len, inner + grp * p.N, p.N, tid, NT);
-        ssd_keep(p, ring, t0, len, inner + p.G * p.N + grp * p.N, p.N, tid, NT);
+        const int inner = p.H * p.P, q0 = p.cu_q[r], ql = p.cu_q[r + 1] - q0;
+        ssd_keep(p, ring, q0, ql, inner + grp * p.N, p.N, tid, NT);
+        ssd_keep(p, ring, q0, ql, inner + p.G * p.N + grp * p.N, p.N, tid, NT);
+    }
+}
+
+// A request's segments in order: carry[item] becomes the state the segment starts from.
+__global__ void __launch_bounds__(256)
+ssd_carry_kernel(const SsdArgs p, const SsdSegments seg) {
+    pdl_wait();
+    const int r = blockIdx.z, h = blockIdx.y, items = seg.items[r], i0 = seg.item0[r], per = p.P * p.N;
+    const int e = blockIdx.x * blockDim.x + threadIdx.x;
+    if (items < 2 || e >= per) return;
+    float S = p.state[(size_t)p.slots[r] * p.slot_stride + (size_t)h * per + e];
+    for (int k = 0; k < items; ++k) {
+        float* at = seg.carry + ((size_t)(i0 + k) * p.H + h) * per + e;
+        if (k + 1 < items) {
+            const float local = *at;
+            *at = S;
+            S = expf(seg.decay[(size_t)(i0 + k) * p.H + h]) * S + local;
+        } else {
+            *at = S;
+        }
     }
 }
 
@@ -719,36 +833,49 @@ static int ssd_run_step(const SsdArgs& p, const TA* xbc, long long ldx, const fl
     return (int)cudaErrorInvalidValue;
 }
 
-template <int NK, int W>
-static int ssd_run_chunk_w(const SsdArgs& p, const bf16* xbc, long long ldx, const float* dts, int n, int n_requests, bf16* out,
-                           long long ldo, cudaStream_t stream) {
-    constexpr size_t smem = SsdTile<NK>::bytes(W);
+template <int NK, int PW, int PASS>
+static int ssd_run_pass(const SsdArgs& p, const bf16* xbc, long long ldx, const float* dts, int n, int items, bf16* out, long long ldo,
+                        const SsdSegments& seg, cudaStream_t stream) {
+    using Tile = SsdTile<NK, PW>;
     static bool raised = false;
     if (!raised) {
-        const cudaError_t e = cudaFuncSetAttribute(ssd_chunk_kernel<NK, W>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        const cudaError_t e = cudaFuncSetAttribute(ssd_chunk_kernel<NK, PW, PASS>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                                   (int)Tile::bytes);
         if (e != cudaSuccess) return (int)e;
         raised = true;
     }
-    const int tiles = (p.P + 16 * W - 1) / (16 * W);
-    return rllm_launch(ssd_chunk_kernel<NK, W>, dim3(p.H * tiles, n_requests), dim3(32 * W), smem, stream, p, xbc, ldx, dts, n, out,
-                       ldo);
+    const int tiles = (p.P + 16 * PW - 1) / (16 * PW);
+    return rllm_launch(ssd_chunk_kernel<NK, PW, PASS>, dim3(p.H * tiles, items), dim3(Tile::NT), Tile::bytes, stream, p, xbc, ldx, dts, n,
+                       out, ldo, seg);
+}
+template <int NK, int PW>
+static int ssd_run_chunk_w(const SsdArgs& p, const bf16* xbc, long long ldx, const float* dts, int n, int n_requests, bf16* out,
+                           long long ldo, const SsdSegments& seg, int n_items, cudaStream_t stream) {
+    if (n_items <= 0) return ssd_run_pass<NK, PW, 0>(p, xbc, ldx, dts, n, n_requests, out, ldo, seg, stream);
+    int st = ssd_run_pass<NK, PW, 1>(p, xbc, ldx, dts, n, n_items, out, ldo, seg, stream);
+    if (st) return st;
+    st = rllm_launch(ssd_carry_kernel, dim3((p.P * p.N + 255) / 256, p.H, n_requests), dim3(256), 0, stream, p, seg);
+    if (st) return st;
+    return ssd_run_pass<NK, PW, 2>(p, xbc, ldx, dts, n, n_items, out, ldo, seg, stream);
 }
 template <int NK>
 static int ssd_run_chunk(const SsdArgs& p, const bf16* xbc, long long ldx, const float* dts, int n, int n_requests, bf16* out,
-                         long long ldo, cudaStream_t stream) {
-    if (p.P <= 16) return ssd_run_chunk_w<NK, 1>(p, xbc, ldx, dts, n, n_requests, out, ldo, stream);
-    if (p.P <= 32) return ssd_run_chunk_w<NK, 2>(p, xbc, ldx, dts, n, n_requests, out, ldo, stream);
-    return ssd_run_chunk_w<NK, 4>(p, xbc, ldx, dts, n, n_requests, out, ldo, stream);
+                         long long ldo, const SsdSegments& seg, int n_items, cudaStream_t stream) {
+    if (p.P <= 16) return ssd_run_chunk_w<NK, 1>(p, xbc, ldx, dts, n, n_requests, out, ldo, seg, n_items, stream);
+    if (p.P <= 32) return ssd_run_chunk_w<NK, 2>(p, xbc, ldx, dts, n, n_requests, out, ldo, seg, n_items, stream);
+    return ssd_run_chunk_w<NK, 4>(p, xbc, ldx, dts, n, n_requests, out, ldo, seg, n_items, stream);
 }
 
 // mode 0: a step of at most SSD_STEP tokens a request, everything in one kernel; 1: portions, token by token; 2: portions
 // (bfloat16, N up to 256) in chunks.  xbc [n, H * P8 + 2 G * N8] (activation type) and dts [2, H, n]: scratch of modes 1 and 2.
-// out (activation type, rows ldo apart): y * silu(z), before the norm.
+// out (activation type, rows ldo apart): y * silu(z), before the norm.  seg_*, n_items: the step's requests cut along time (mode 2;
+// n_items 0: not cut), carry [n_items, H, P, N] and decay [n_items, H] scratch.
 RLLM_API int rllm_ssd(const float* rows, long long ld, int z_off, int c_off, int dt_off, const float* conv, const float* conv_b,
                       const float* dt_bias, const float* A, const float* D, float* state, long long slot_stride,
                       const int* positions, const int* seq_ids, const int* cu_q, const int* slots, int H, int G, int P, int N,
                       int taps, int n, int n_requests, int mode, void* xbc, long long ldx, float* dts, void* out, int out_dt,
-                      long long ldo, cudaStream_t stream) {
+                      long long ldo, const int* seg_t0, const int* seg_t1, const int* seg_req, const int* seg_flags,
+                      const int* req_item0, const int* req_items, int n_items, float* carry, float* decay, cudaStream_t stream) {
     if (n <= 0) return 0;
     if (H <= 0 || G <= 0 || H % G || P <= 0 || N <= 0 || taps < 1 || n_requests <= 0 || mode < 0 || mode > 2 ||
         (mode > 0 && (!xbc || !dts || ldx < (long long)H * ssd_pad8(P) + 2LL * G * ssd_pad8(N))))
@@ -765,11 +892,16 @@ RLLM_API int rllm_ssd(const float* rows, long long ld, int z_off, int c_off, int
             ? ssd_run_step<float>(p, (const float*)xbc, ldx, dts, n, n_requests, (float*)out, ldo, mode == 0, stream)
             : ssd_run_step<bf16>(p, (const bf16*)xbc, ldx, dts, n, n_requests, (bf16*)out, ldo, mode == 0, stream);
     if (out_dt != RLLM_BF16 || N > 256 || ldx % 8 || ((uintptr_t)xbc & 15)) return (int)cudaErrorInvalidValue;
+    if (n_items > 0 && (!seg_t0 || !seg_t1 || !seg_req || !seg_flags || !req_item0 || !req_items || !carry || !decay))
+        return (int)cudaErrorInvalidValue;
     const bf16* x = (const bf16*)xbc;
-    if (N <= 32) return ssd_run_chunk<2>(p, x, ldx, dts, n, n_requests, (bf16*)out, ldo, stream);
-    if (N <= 64) return ssd_run_chunk<4>(p, x, ldx, dts, n, n_requests, (bf16*)out, ldo, stream);
-    if (N <= 128) return ssd_run_chunk<8>(p, x, ldx, dts, n, n_requests, (bf16*)out, ldo, stream);
-    return ssd_run_chunk<16>(p, x, ldx, dts, n, n_requests, (bf16*)out, ldo, stream);
+    const SsdSegments seg = {seg_t0, seg_t1, seg_req, seg_flags, req_item0, req_items, carry, decay};
+#define SSD_CHUNKS(NK) return ssd_run_chunk<NK>(p, x, ldx, dts, n, n_requests, (bf16*)out, ldo, seg, n_items, stream)
+    if (N <= 32) SSD_CHUNKS(2);
+    if (N <= 64) SSD_CHUNKS(4);
+    if (N <= 128) SSD_CHUNKS(8);
+    SSD_CHUNKS(16);
+#undef SSD_CHUNKS
 }
 
 RLLM_API int rllm_ssd_norm(void* v, int dt, long long ld, const float* w, int n, int parts, int size, float eps,

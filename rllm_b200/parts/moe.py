@@ -30,8 +30,8 @@ and weights are float32 in every mode.
 
 Steps of few rows run every (token, chosen expert) pair against its expert's matrices directly, with no
 host involvement (so such steps can be captured into graphs).  Steps of many rows sort the pairs by
-expert on the device, read the experts' counts back and run each expert's rows through the package's
-products.
+expert on the device; experts without a gate then run as two grouped products (one launch each, no host involvement), gated
+ones, float32 and odd sizes by reading the experts' counts back and running each expert's rows through the package's products.
 """
 from __future__ import annotations
 
@@ -132,16 +132,19 @@ class RoutedExperts(FeedForward):
         n, d, dev, dt = h.shape[0], self.hidden_size, h.device, self.runtime.dtype
         idx, weight, logits = self.route(h)
         shared = gate = None
+        few = n <= PAIR_ROWS or torch.cuda.is_current_stream_capturing()
         if self.shared_size:
             act = torch.empty((n, self.shared_size), dtype=dt, device=dev)
-            if self.activation is not None:
+            if self.activation is not None and not few and ops.gemm_group_ok(h, self.w_shared_gu):
+                ops.gemm_group(h, self.w_shared_gu, act, activation=self.activation)       # the activation in the product's epilogue
+            elif self.activation is not None:
                 ops.rows_act(ops.linear(h, self.w_shared_gu, out_dtype=torch.float32), act, act=self.activation)
             else:
                 ops.gate_up_swiglu(h, self.w_shared_gu, act, glu=self.shared_form)
             shared = ops.linear(act, self.w_shared_down, out_dtype=torch.float32)
             gate = logits[:, self.E:self.E + 1] if self.shared_gate else None
         out = torch.empty((n, d), dtype=torch.float32, device=dev)
-        if n <= PAIR_ROWS or torch.cuda.is_current_stream_capturing():
+        if few:
             act = torch.empty((n * self.top_k, self.F), dtype=dt, device=dev)
             if self.activation is not None:
                 ops.moe_pairs_up(h, self.w_gu, idx, weight if self.weigh_input else None, act, self.activation)
@@ -155,9 +158,14 @@ class RoutedExperts(FeedForward):
         rows = torch.empty((n * self.top_k, d), dtype=dt, device=dev)
         w_rows = torch.empty(n * self.top_k, dtype=torch.float32, device=dev) if self.weigh_input else None
         ops.moe_gather_rows(h, place, rows, self.top_k, weight if self.weigh_input else None, w_rows)
-        bounds = offsets.tolist()                          # the host learns how many rows each expert has
         act = torch.empty((n * self.top_k, self.F), dtype=dt, device=dev)
         y = torch.empty((n * self.top_k, d), dtype=torch.float32, device=dev)
+        if self.activation is not None and ops.gemm_group_ok(rows, self.w_gu) and ops.gemm_group_ok(act, self.w_down):
+            # all experts in one launch each, the tiles counted from the offsets on the device
+            ops.gemm_group(rows, self.w_gu, act, offsets, row_scale=w_rows, activation=self.activation)
+            ops.gemm_group(act, self.w_down, y, offsets)
+            return ops.moe_combine(y, place, None if self.weigh_input else weight, out, shared, gate, self.top_k)
+        bounds = offsets.tolist()                          # the host learns how many rows each expert has
         if self.activation is not None:
             up = torch.empty((n * self.top_k, self.F), dtype=torch.float32, device=dev)
             for e in range(self.E):

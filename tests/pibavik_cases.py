@@ -74,7 +74,7 @@ CASES = {
     # head sizes of 64 and 128 take the tensor-core attention kernels in bfloat16
     "heads64": config([sloped(8, 2, 64, 64, 21, 0.12, moe(48, 8, 2, 40)), sloped(8, 2, 64, 64, 70, 0.12, None, 0),
                        parallel((4, 2, 64, 64, 33, 0.15), (16, 50000.0), (4, 64, 64, 2, 4, 4), moe(32, 8, 1))], width=64, vocab=113),
-    "heads128": config([sloped(3, 1, 128, 128, 50, 0.1), parallel((2, 2, 128, 128, 40, 0.1), (128, 10000.0), (3, 32, 128, 1, 4, 1)),
+    "heads128": config([sloped(3, 1, 128, 128, 34, 0.1), parallel((2, 2, 128, 128, 40, 0.1), (128, 10000.0), (3, 32, 128, 1, 4, 1)),
                         latent(4, 64, 48, 72, 128, 0.12, moe(40, 4, 2))], width=56, vocab=103),
     # sizes that are no multiple of 2, 4 or 8 wherever the design allows it
     "odd_sizes": config([sloped(3, 1, 7, 5, 6, 0.7, moe(9, 5, 2, 11)), parallel((3, 1, 9, 11, 4, 0.5), (6, 99.0), (5, 7, 3, 5, 3, 5), moe(7, 3, 1)),
