@@ -45,7 +45,8 @@ template <typename TC> __device__ __forceinline__ void gg_store32(TC* dst, const
     }
 }
 
-template <typename TC>
+// ACT: the activation's number, or -1: `act` decides (a switch per element in the epilogue's loop costs more than the products)
+template <typename TC, int ACT>
 __global__ void __launch_bounds__(GG_THREADS, 1)
 gemm_group_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUtensorMap tmB, TC* C, long long ldc, const int* offsets,
                   int E, int rows, int N, int K, const float* row_scale, int act, int* err) {
@@ -203,16 +204,8 @@ gemm_group_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant
                 }
                 const int gn = n0 + c0;
                 if (gm < m_end && gn < N) {
-                    if (act == ACT_RELU2) {
 #pragma unroll
-                        for (int j = 0; j < 32; ++j) {
-                            const float z = fmaxf(scale * __uint_as_float(r[j]), 0.f);
-                            v[j] = z * z;
-                        }
-                    } else {
-#pragma unroll
-                        for (int j = 0; j < 32; ++j) v[j] = act_apply(scale * __uint_as_float(r[j]), act);
-                    }
+                    for (int j = 0; j < 32; ++j) v[j] = act_apply(scale * __uint_as_float(r[j]), ACT >= 0 ? ACT : act);
                     gg_store32<TC>(C + (size_t)gm * ldc + gn, v, min(32, N - gn));
                 }
             }
@@ -247,15 +240,11 @@ RLLM_API int rllm_gemm_group(const void* A, const void* B, void* C, int c_dtype,
     st = gg_tmap(&tb, B, (long long)E * N, K, GG_BN);
     if (st) return st;
     constexpr int smem = GG_STAGES * (GG_BM + GG_BN) * GG_BK * 2 + 1024;
-    auto kf = gemm_group_kernel<float>;
-    auto kb = gemm_group_kernel<bf16>;
-    static bool attr_set = false;
-    if (!attr_set) {
-        cudaError_t e = cudaFuncSetAttribute(kf, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
-        if (e == cudaSuccess) e = cudaFuncSetAttribute(kb, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    auto run = [&](auto kern, auto* out, int grid) -> int {
+        const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
         if (e != cudaSuccess) return (int)e;
-        attr_set = true;
-    }
+        return rllm_launch(kern, dim3(grid), dim3(GG_THREADS), smem, stream, ta, tb, out, ldc, offsets, E, rows, N, K, row_scale, act, err);
+    };
     static int n_sm = 0;
     if (!n_sm) {
         int dev = 0;
@@ -264,10 +253,14 @@ RLLM_API int rllm_gemm_group(const void* A, const void* B, void* C, int c_dtype,
         if (n_sm <= 0) n_sm = 148;
     }
     const long long most = ((long long)(rows + GG_BM - 1) / GG_BM + (offsets ? E : 0)) * ((N + GG_BN - 1) / GG_BN);
-    const dim3 grid((unsigned)(most < n_sm ? most : n_sm));
-    if (c_dtype == RLLM_F32)
-        return rllm_launch(kf, grid, dim3(GG_THREADS), smem, stream, ta, tb, (float*)C, ldc, offsets, E, rows, N, K, row_scale, act, err);
-    return rllm_launch(kb, grid, dim3(GG_THREADS), smem, stream, ta, tb, (bf16*)C, ldc, offsets, E, rows, N, K, row_scale, act, err);
+    const int grid = (int)(most < n_sm ? most : n_sm);
+#define GG_RUN(T)                                                                          \
+    if (act == ACT_NONE) return run(gemm_group_kernel<T, ACT_NONE>, (T*)C, grid);          \
+    if (act == ACT_RELU2) return run(gemm_group_kernel<T, ACT_RELU2>, (T*)C, grid);        \
+    return run(gemm_group_kernel<T, -1>, (T*)C, grid);
+    if (c_dtype == RLLM_F32) { GG_RUN(float) }
+    GG_RUN(bf16)
+#undef GG_RUN
 }
 
 TC_DEFINE_WAIT_CONTROLS(rllm_gemm_group)

@@ -1109,7 +1109,7 @@ def ssd(rows, conv, conv_b, dt_bias, A, D, norm_w, eps, norm_groups, state, ctx,
                                      c_int(norm_groups), c_int(inner // norm_groups), c_float(eps), _stream()), "ssd_norm")
     if mode:
         global _launches
-        _launches += 3 if sg is not None else 1      # the convolution's kernel, the local pass and the carry
+        _launches += 2 if sg is not None else 1      # the convolution's kernel, the pass ahead of a cut portion's
     return out
 
 

@@ -22,8 +22,8 @@
 //   ssd_chunk   bfloat16 portions on the tensor cores, in chunks of 64 tokens counted from the portion's start: a block
 //               per (head, 16 to 64 rows of S, request) walks the request's chunks with S^T in the accumulators of
 //               mma.sync (two warps, the halves of N, per 16 rows).  Long portions are also cut along time: pass 1 works
-//               out what every segment's tokens leave from an empty state, ssd_carry the state that every segment starts
-//               from, pass 2 the outputs, all segments side by side.  With L_i = log(a_1 .. a_i) of a chunk:
+//               out what every segment's tokens leave, pass 2 the outputs from the states that follow, all segments side
+//               by side.  With L_i = log(a_1 .. a_i) of a chunk:
 //                   y_i = e^(L_i) S0 C_i + sum_(j<=i) (C_i . B_j) e^(L_i - L_j) d_j x_j
 //                   S   = e^(L_64) S0 + sum_j e^(L_64 - L_j) d_j x_j B_j^T
 //               x, B and C are bfloat16 as stored; every other operand (S0, the weighted scores, the weighted x) goes into
@@ -57,11 +57,6 @@ __device__ __forceinline__ int ssd_channels(const SsdArgs& p) { return p.H * p.P
 __device__ __forceinline__ int ssd_ring(const SsdArgs& p) { return p.taps - 1 + SSD_STEP; }
 __host__ __device__ __forceinline__ int ssd_pad8(int n) { return (n + 7) / 8 * 8; }
 
-// the input of channel c `back` tokens before the flat token t (the request's token i, at position pos)
-__device__ __forceinline__ float ssd_input(const SsdArgs& p, const float* ring, int t, int i, int pos, int back, int c) {
-    if (back <= i) return p.rows[(size_t)(t - back) * p.ld + p.c_off + c];
-    return back <= pos ? ring[(size_t)((pos - back) % ssd_ring(p)) * ssd_channels(p) + c] : 0.f;
-}
 // The ring entries of the request's last tokens, for the channels c0 .. c0 + count - 1.
 __device__ __forceinline__ void ssd_keep(const SsdArgs& p, float* ring, int t0, int len, int c0, int count, int tid, int nt) {
     const int m = min(len, p.taps - 1), C = ssd_channels(p), R = ssd_ring(p);
@@ -238,6 +233,8 @@ ssd_step_kernel(const SsdArgs p, const TA* xbc, long long ldx, const float* dts,
         const int cnt = min(SSD_STEP, len - c0);
         load(grp);                                   // on its way while the convolutions run
         const int per = p.P + 2 * p.N;
+        float z_first = 0.f;                         // the gate of the thread's first output, on its way
+        if (tid < cnt * p.P) z_first = p.rows[(size_t)(t0 + c0 + tid / p.P) * p.ld + p.z_off + (size_t)h * p.P + tid % p.P];
         for (int e = tid; e < cnt * per; e += blockDim.x) {
             const int i = e / per, c = e - i * per, t = t0 + c0 + i;
             float v;
@@ -245,7 +242,20 @@ ssd_step_kernel(const SsdArgs p, const TA* xbc, long long ldx, const float* dts,
                 const int ch = c < p.P ? h * p.P + c : c < p.P + p.N ? inner + g * p.N + c - p.P : inner + gn + g * p.N + c - p.P - p.N;
                 const int C = ssd_channels(p), pos = p.positions[t];
                 float acc = p.conv_b[ch];
-                for (int j = 0; j < p.taps; ++j) acc += p.conv[(size_t)j * C + ch] * ssd_input(p, ring, t, i, pos, p.taps - 1 - j, ch);
+                for (int j0 = 0; j0 < p.taps; j0 += 4) {          // four inputs and their weights in flight
+                    float in[4], w[4];
+#pragma unroll
+                    for (int j = 0; j < 4; ++j) {
+                        const int back = p.taps - 1 - j0 - j;
+                        const float* at = back <= i ? p.rows + (size_t)(t - back) * p.ld + p.c_off + ch
+                                                    : ring + (size_t)((pos - back + ssd_ring(p)) % ssd_ring(p)) * C + ch;
+                        const bool ok = back >= 0 && back <= pos;
+                        in[j] = ok ? *at : 0.f;
+                        w[j] = back >= 0 ? p.conv[(size_t)(j0 + j) * C + ch] : 0.f;
+                    }
+#pragma unroll
+                    for (int j = 0; j < 4; ++j) acc += w[j] * in[j];
+                }
                 v = to_f<TA>(from_f<TA>(silu_f(acc)));          // as stored where a kernel of its own does this
             } else {
                 const int col = c < p.P ? h * P8 + c : c < p.P + p.N ? p.H * P8 + g * N8 + c - p.P
@@ -330,7 +340,7 @@ ssd_step_kernel(const SsdArgs p, const TA* xbc, long long ldx, const float* dts,
         for (int e = tid; e < cnt * p.P; e += blockDim.x) {
             const int i = e / p.P, c = e - i * p.P;
             const size_t t = t0 + c0 + i;
-            const float z = p.rows[t * p.ld + p.z_off + (size_t)h * p.P + c];
+            const float z = e == tid ? z_first : p.rows[t * p.ld + p.z_off + (size_t)h * p.P + c];
             out[t * ldo + (size_t)h * p.P + c] = from_f<TA>((s_y[e] + Dh * s_x[e]) * silu_f(z));
         }
         __syncthreads();
@@ -378,7 +388,8 @@ struct SsdSegments {
     const int* flags;     // [items] bit 0: first segment of its request, bit 1: last
     const int* item0;     // [requests] a request's first item
     const int* items;     // [requests] how many it has
-    float* carry;         // [items][H][P][N]: what a segment's tokens leave from an empty state, then the state it starts from
+    float* carry;         // [items][H][P][N], of a request with several: the state behind its first segment, what the tokens of a
+                          // middle one leave from an empty state, and (at its last) the state it came with
     float* decay;         // [items][H]: the sum of the segment's log decays
 };
 
@@ -393,8 +404,8 @@ template <int NK, int PW> struct SsdTile {           // N padded to 16 * NK, 16 
     static constexpr size_t bytes = 2 * stage + (m_bytes > y_bytes ? m_bytes : y_bytes) + 2 * 2 * SSD_CHUNK * sizeof(float);
 };
 
-// PASS 0: whole requests.  1: what the tokens of a segment leave from an empty state, and their decay; no output.  2: segments
-// from the state they start from, with output.
+// PASS 0: whole requests.  1: what SsdSegments says of carry, and a segment's decay; no output.  2: segments from the state they
+// start from (put together from carry: the blocks of a request's last segment overwrite its slot), with output.
 template <int NK, int PW, int PASS>
 __global__ void __launch_bounds__(PW * 64, NK <= 8 ? 8 / PW : 4 / PW)
 ssd_chunk_kernel(const SsdArgs p, const bf16* xbc, long long ldx, const float* dts, int n, bf16* out, long long ldo,
@@ -413,12 +424,17 @@ ssd_chunk_kernel(const SsdArgs p, const bf16* xbc, long long ldx, const float* d
     const int item = blockIdx.y, r = PASS == 0 ? item : seg.req[item];
     const int t0 = PASS == 0 ? p.cu_q[r] : seg.t0[item], len = (PASS == 0 ? p.cu_q[r + 1] : seg.t1[item]) - t0;
     const bool first = PASS == 0 || (seg.flags[item] & 1), last = PASS == 0 || (seg.flags[item] & 2);
-    if (len <= 0 || (PASS == 1 && last)) return;             // a request's last segment leaves its state in pass 2
+    if (len <= 0 || (PASS == 1 && first && last)) return;
     const int grp = h / (p.H / p.G), P8 = ssd_pad8(p.P), N8 = ssd_pad8(p.N);
     float* slot = p.state + (size_t)p.slots[r] * p.slot_stride;
     float* Sg = slot + (size_t)h * p.P * p.N;
-    float* Sc = PASS == 0 ? nullptr : seg.carry + ((size_t)item * p.H + h) * p.P * p.N;
+    float* Sc = PASS == 0 ? nullptr : seg.carry + ((size_t)item * p.H + h) * p.P * p.N;        // (pass 1)
     float* ring = slot + p.ring_base;
+    const int per = p.P * p.N, rows_here = min(16 * PW, p.P - p0);
+    if (PASS == 1 && last) {
+        for (int e = tid; e < rows_here * p.N; e += NT) Sc[(size_t)p0 * p.N + e] = Sg[(size_t)p0 * p.N + e];
+        return;
+    }
 
     const bf16* x_src = xbc + (size_t)t0 * ldx + (size_t)h * P8 + p0;
     const bf16* b_src = xbc + (size_t)t0 * ldx + (size_t)p.H * P8 + (size_t)grp * N8;
@@ -465,14 +481,30 @@ ssd_chunk_kernel(const SsdArgs p, const bf16* xbc, long long ldx, const float* d
     // S^T: rows row0 and row0 + 8 of this lane, columns n0 + 8 j + c2, + 1 (the warp's half of N)
     const int row0 = p0 + pw * 16 + g8, n0 = half * NH * 16;
     float S[2 * NH][4];
-    const float* S_from = (PASS == 2 && !(first && last)) ? Sc : Sg;      // (the slot's own state is what the last segment overwrites)
+    // S <- decay * S + what lies at `from`
+    auto take = [&](const float* from, float decay) {
 #pragma unroll
-    for (int j = 0; j < 2 * NH; ++j)
+        for (int j = 0; j < 2 * NH; ++j)
 #pragma unroll
-        for (int q = 0; q < 4; ++q) {
-            const int row = row0 + (q >> 1) * 8, c = n0 + 8 * j + c2 + (q & 1);
-            S[j][q] = PASS != 1 && row < p.P && c < p.N ? S_from[(size_t)row * p.N + c] : 0.f;
+            for (int q = 0; q < 4; ++q) {
+                const int row = row0 + (q >> 1) * 8, c = n0 + 8 * j + c2 + (q & 1);
+                S[j][q] = decay * S[j][q] + (row < p.P && c < p.N ? from[(size_t)row * p.N + c] : 0.f);
+            }
+    };
+#pragma unroll
+    for (int j = 0; j < 2 * NH; ++j) S[j][0] = S[j][1] = S[j][2] = S[j][3] = 0.f;
+    if (PASS != 2 || (first && last)) {
+        if (PASS != 1 || first) take(Sg, 0.f);
+    } else {
+        const int i0 = seg.item0[r];
+        auto at = [&](int i) { return seg.carry + ((size_t)i * p.H + h) * per; };
+        if (first) {
+            take(at(i0 + seg.items[r] - 1), 0.f);
+        } else {
+            take(at(i0), 0.f);
+            for (int i = i0 + 1; i < item; ++i) take(at(i), expf(seg.decay[(size_t)i * p.H + h]));
         }
+    }
     const float Dh = p.D[h];
     const bool vec = p.P % 8 == 0 && p.ld % 4 == 0 && p.z_off % 4 == 0 && ldo % 8 == 0 && ((uintptr_t)p.rows & 15) == 0 &&
                      ((uintptr_t)out & 15) == 0;
@@ -702,26 +734,6 @@ ssd_chunk_kernel(const SsdArgs p, const bf16* xbc, long long ldx, const float* d
     }
 }
 
-// A request's segments in order: carry[item] becomes the state the segment starts from.
-__global__ void __launch_bounds__(256)
-ssd_carry_kernel(const SsdArgs p, const SsdSegments seg) {
-    pdl_wait();
-    const int r = blockIdx.z, h = blockIdx.y, items = seg.items[r], i0 = seg.item0[r], per = p.P * p.N;
-    const int e = blockIdx.x * blockDim.x + threadIdx.x;
-    if (items < 2 || e >= per) return;
-    float S = p.state[(size_t)p.slots[r] * p.slot_stride + (size_t)h * per + e];
-    for (int k = 0; k < items; ++k) {
-        float* at = seg.carry + ((size_t)(i0 + k) * p.H + h) * per + e;
-        if (k + 1 < items) {
-            const float local = *at;
-            *at = S;
-            S = expf(seg.decay[(size_t)(i0 + k) * p.H + h]) * S + local;
-        } else {
-            *at = S;
-        }
-    }
-}
-
 // ------------------------------------------------------------------ norm of the gated rows
 // One block per (token, part): v[t, part] /= rms(v[t, part]), times w; in place.
 template <typename T, int VEC>
@@ -852,9 +864,7 @@ template <int NK, int PW>
 static int ssd_run_chunk_w(const SsdArgs& p, const bf16* xbc, long long ldx, const float* dts, int n, int n_requests, bf16* out,
                            long long ldo, const SsdSegments& seg, int n_items, cudaStream_t stream) {
     if (n_items <= 0) return ssd_run_pass<NK, PW, 0>(p, xbc, ldx, dts, n, n_requests, out, ldo, seg, stream);
-    int st = ssd_run_pass<NK, PW, 1>(p, xbc, ldx, dts, n, n_items, out, ldo, seg, stream);
-    if (st) return st;
-    st = rllm_launch(ssd_carry_kernel, dim3((p.P * p.N + 255) / 256, p.H, n_requests), dim3(256), 0, stream, p, seg);
+    const int st = ssd_run_pass<NK, PW, 1>(p, xbc, ldx, dts, n, n_items, out, ldo, seg, stream);
     if (st) return st;
     return ssd_run_pass<NK, PW, 2>(p, xbc, ldx, dts, n, n_items, out, ldo, seg, stream);
 }
