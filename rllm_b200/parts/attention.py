@@ -69,8 +69,9 @@ class Attention(Mixer):
                 self.hd_s = self.hdv_s = size
         short = p.get("names") == "short"
         self.plain = self.hdv == self.hd and not self.has_sink and self.own_kv and self.slope_values is None
-        if (self.hd % 16 and self.plain) or (self.hd % 2 and self.slope_values is None) or self.hd > 256 or self.hdv > 256:
-            raise PartError(f"attention: head_dim {self.hd} must be a multiple of 16 and at most 256")
+        most = 256 if self.slope_values is None else 512
+        if (self.hd % 16 and self.plain) or (self.hd % 2 and self.slope_values is None) or max(self.hd, self.hdv) > most:
+            raise PartError(f"attention: head_dim {self.hd} must be a multiple of 16 and at most {most}")
         n = (lambda s: s) if short else (lambda s: {"q.norm": "q_norm.weight", "k.norm": "k_norm.weight",
                                                     "sink": "sink"}.get(s, s + "_proj.weight"))
         self._n = {s: self.prefix + n(s) for s in ("q", "k", "v", "o", "q.norm", "k.norm", "sink")}
