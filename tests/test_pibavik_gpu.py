@@ -284,7 +284,7 @@ def run_ssd(rows, par, state, lens, starts, slots, H, P, N, G, dtype, parts=1, e
     return out
 
 
-SSD_SIZES = [(4, 16, 32, 2, 4, 2), (6, 32, 48, 2, 4, 3), (2, 64, 128, 1, 4, 1), (3, 7, 5, 3, 3, 7), (4, 24, 16, 1, 1, 4), (2, 80, 64, 2, 2, 1),
+SSD_SIZES = [(4, 16, 32, 2, 4, 2), (6, 40, 56, 3, 4, 4), (2, 64, 128, 1, 4, 1), (3, 7, 5, 3, 3, 7), (4, 24, 16, 1, 1, 4), (2, 80, 64, 2, 2, 1),
              (1, 136, 20, 1, 6, 2), (3, 40, 130, 1, 4, 1), (2, 16, 256, 2, 4, 2), (5, 12, 9, 5, 5, 6), (8, 64, 64, 8, 4, 8), (2, 1, 3, 1, 4, 1)]
 
 
